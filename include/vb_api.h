@@ -527,7 +527,7 @@ int vb_postnorm_residual_f32(float* d_x, const float* d_y, int y_planes, const f
 int vb_linear(void* d_out, const void* d_x, const void* d_w, int T, int N, int K, int ldx, int ldo, int in_dtype,
               int out_dtype, int epilogue, float alpha, const int32_t* d_row_off, const int32_t* d_gather, int groups,
               long long w_group_stride, float glu_limit, float glu_slope, void* stream);
-/* (vb_linear epilogues 2, 3, 4: relu(y)^2, gelu (erf), gelu (tanh).  Epilogue 1 with glu_limit > 0 is the clamped gated
+/* (vb_linear epilogues 2, 3, 4: relu(y)^2, gelu (erf), gelu (tanh); 5: gate and up rows as 1, gelu(gate) (tanh) * up.  Epilogue 1 with glu_limit > 0 is the clamped gated
  * form: g = min(gate, limit), u = clamp(up, -limit, limit), Y = g * sigmoid(glu_slope * g) * (u + 1).)
  * vb_linear_batched: `groups` independent products that share their rows (the heads of a token side by side): group g reads
  * X + g * x_group_stride, W + g * w_group_stride and writes Y + g * o_group_stride, all with T rows; with d_gate,
@@ -558,7 +558,9 @@ int vb_rotary_table(float* d_cs, const int32_t* d_pos, const double* d_freq, int
  * vb_qkv_norm_rotary_append: like vb_qkv_rotary_append for heads that are RMS-normed over their dim values before the
  *   rotation (d_q_norm / d_k_norm [dim], shared by all heads; NULL: no norm); layout 0 rotates pairs (2i, 2i + 1), layout 1
  *   pairs (i, i + half).  Hq query heads, Gk key heads [pages][page][Gk][dim], Gv value heads [pages][page][Gv][vdim]
- *   (attention with several score maps per head counts every map as a head: Gk = maps * Gv).
+ *   (attention with several score maps per head counts every map as a head: Gk = maps * Gv).  d_bias (optional; q, k, v
+ *   columns side by side): one value per column of the projection row, added first; d_q_scale [Hq] (optional): every query
+ *   head times its factor, last; v_norm: every value head is divided by sqrt(mean(v^2) + eps).
  * vb_latent_rope_append: tail of a fused (queries | latent + shared rotated key part) projection: heads of `dim` unrotated +
  *   `rot` rotated dims.  The latent is RMS-normed (d_wc) and appended with the rotated key part as ONE row [kv_rank | rot]
  *   of d_cache; the queries' unrotated parts go to d_q_out [T][H][dim], their rotated parts to
@@ -569,7 +571,8 @@ int vb_qkv_norm_rotary_append(const float* d_proj, int ldp, int q_off, int k_off
                               int layout, const float* d_q_norm, const float* d_k_norm, float eps, void* d_q_out,
                               void* d_k_cache, void* d_v_cache, const int32_t* d_row_req, const int32_t* d_pos,
                               const int32_t* d_page_indptr, const int32_t* d_page_indices, int page_size, int T, int Hq, int Gk,
-                              int Gv, int dim, int vdim, int dtype, void* stream);
+                              int Gv, int dim, int vdim, int dtype, const float* d_bias, const float* d_q_scale, int v_norm,
+                              void* stream);
 int vb_latent_rope_append(const float* d_proj, int ldp, int q_off, int c_off, int H, int dim, int rot, int kv_rank,
                           const float* d_wc, const float* d_cs, int half, int layout, void* d_q_out, void* d_q_lat,
                           void* d_cache, const int32_t* d_row_req, const int32_t* d_pos, const int32_t* d_page_indptr,
@@ -588,22 +591,25 @@ int vb_qkv_rotary_append(const float* d_proj, int ldp, int q_off, int k_off, int
 int vb_latent_norm_append(const float* d_proj, int ldp, int q_off, int c_off, int q_rank, int kv_rank, const float* d_wq,
                           const float* d_wc, void* d_cq_out, void* d_c_cache, const int32_t* d_row_req, const int32_t* d_pos,
                           const int32_t* d_page_indptr, const int32_t* d_page_indices, int page_size, int T, float eps,
-                          int dtype, void* stream);
+                          int rot, const float* d_cs, int half, int layout, int dtype, void* stream);
+/* (rot > 0: the latent's columns are followed by a key part of `rot` dims shared by all heads, whose first 2 * half dims are
+ * rotated; d_c_cache then holds rows [kv_rank | rot].) */
 int vb_window_attn(void* d_out, const void* d_q, const void* d_k_cache, const void* d_v_cache, const float* d_gate,
                    int ld_gate, const int32_t* d_row_req, const int32_t* d_pos, const int32_t* d_page_indptr,
                    const int32_t* d_page_indices, int T, int H, int G, int dim, int vdim, int page_size, int window,
                    float scale, int dtype, float* d_part, long long part_floats, const int32_t* d_row_list, int head_rows,
-                   int chunk, int k_ld, int v_ld, int v_share, int out_f32, void* stream);
+                   int chunk, int k_ld, int v_ld, int v_share, int out_f32, const float* d_sink, void* stream);
 /* (chunk > 0: a position sees only the keys of its own block of `chunk` positions, counted from position 0.  k_ld / v_ld:
  * elements per token of the key / value cache (<= 0: G * dim, (G / v_share) * vdim); a value that is a leading slice of
  * the single key head has v_ld = k_ld and the same base pointer.  v_share consecutive key heads read one value head.
- * out_f32: the output is fp32 [T][H * vdim] whatever the operand type.) */
+ * out_f32: the output is fp32 [T][H * vdim] whatever the operand type.  d_sink [H] (optional): the denominator of head h's
+ * softmax has exp(d_sink[h]) added, a further key of that score without a value.) */
 int vb_window_attn_tile_rows(void);
 int vb_window_attn_tiled(void* d_out, const void* d_q, const void* d_k_cache, const void* d_v_cache, const float* d_gate,
                          int ld_gate, const int32_t* d_pos, const int32_t* d_page_indptr, const int32_t* d_page_indices,
                          const int32_t* d_qo_indptr, const int32_t* d_tile_req, const int32_t* d_tile_row0, int n_tiles,
                          int T, int H, int G, int dim, int vdim, int page_size, int window, float scale, int dtype,
-                         int chunk, int k_ld, int v_ld, int v_share, int out_f32, void* stream);
+                         int chunk, int k_ld, int v_ld, int v_share, int out_f32, const float* d_sink, void* stream);
 /* Element-wise gated recurrence (minGRU) over fp32 state slots [slots][width]: z = sigmoid(pz + bz), u = px + bx,
  * c = u + 1/2 (u >= 0) or sigmoid(u), S_t = (1 - z) S_(t-1) + z c (S = 0 before position 0), out = S_t * silu(pg); pz, px,
  * pg are columns z_off, x_off, g_off of the fp32 projection rows.  single_rows / multi_rows select the requests served.
@@ -705,6 +711,16 @@ int vb_short_conv(void* d_out, int ld_out, float* d_out_f32, int ld_f32, const f
                   const float* d_bias, float* d_state, const int32_t* d_qo_indptr, const int32_t* d_row_req, const int32_t* d_pos,
                   const int32_t* d_slots, int T, int B, int channels, int taps, int act, int residual, int out_dtype,
                   void* stream);
+/* Hyper-connections (hyper.cu): a residual stream of `streams` copies d_xs [T][streams][width] (fp32, in place).
+ *   x_t <- sum_s d_mix[s][t] x_s + d_out_c[t] (d_y + d_bias) (d_x0 given: every copy starts as that row instead; keep_streams
+ *   == 0: the new copies are not written back), u = sum_s d_in_c[s] x_s (NULL: coefficients of one), then
+ *   d_w given:  h = u / sqrt(mean(u^2) + eps) * d_w to d_h (operand type) and / or d_h32 (fp32);  d_w NULL: d_h32 = u.
+ *   d_conv_w [width][taps] (steps in which row t is the only row of request t; taps <= 4): h <- h + conv(h), the causal
+ *   convolution of vb_short_conv on the slot d_slots[t] of d_conv_state [slots][taps - 1][width], which takes h. */
+int vb_hyper_mix_norm(float* d_xs, int streams, const float* d_x0, const float* d_y, const float* d_bias, const float* d_mix,
+                      const float* d_out_c, const float* d_in_c, const float* d_w, void* d_h, float* d_h32, int T, int width,
+                      float eps, const float* d_conv_w, int taps, float* d_conv_state, const int32_t* d_pos,
+                      const int32_t* d_slots, int keep_streams, int out_dtype, void* stream);
 int vb_cast_rows(void* d_out, const float* d_in, int ld_in, int T, int n, int out_dtype, void* stream);
 int vb_qk_norm_append(const float* d_proj, int ldp, int q_off, int k_off, int v_off, const float* d_q_norm,
                       const float* d_k_norm, float eps, void* d_q_out, void* d_k_cache, void* d_v_cache,

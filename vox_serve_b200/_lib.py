@@ -112,7 +112,7 @@ SIGNATURES = {
     "vb_linear_batched": (c_int, [P, P, P, c_int, c_int, c_int, c_int, c_int, C.c_longlong, C.c_longlong, C.c_longlong, c_int,
                                   c_int, c_int, c_int, c_float, P, c_int, P]),
     "vb_latent_norm_append": (c_int, [P, c_int, c_int, c_int, c_int, c_int, P, P, P, P, P, P, P, P, c_int, c_int, c_float,
-                                      c_int, P]),
+                                      c_int, P, c_int, c_int, c_int, P]),
     "vb_moe_route_sigmoid": (c_int, [P, P, P, P, P, P, P, c_int, c_int, c_int, c_int, c_int, c_int, c_int, P]),
     "vb_layernorm_f32": (c_int, [P, P, P, P, P, c_int, c_int, c_float, c_int, P]),
     "vb_postnorm_residual_f32": (c_int, [P, P, c_int, P, P, P, P, P, c_int, c_int, c_float, c_int, P]),
@@ -122,7 +122,7 @@ SIGNATURES = {
     "vb_sum_planes_f32": (c_int, [P, P, c_int, C.c_longlong, P]),
     "vb_rotary_table": (c_int, [P, P, P, c_int, c_int, C.c_double, P]),
     "vb_qkv_norm_rotary_append": (c_int, [P, c_int, c_int, c_int, c_int, P, c_int, c_int, P, P, c_float, P, P, P, P, P, P, P,
-                                          c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, P]),
+                                          c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, P, P, c_int, P]),
     "vb_latent_rope_append": (c_int, [P, c_int, c_int, c_int, c_int, c_int, c_int, c_int, P, P, c_int, c_int, P, P, P, P, P, P,
                                       P, c_int, c_int, c_float, c_int, P]),
     "vb_head_pair_combine": (c_int, [P, P, P, c_int, c_int, c_int, c_int, c_int, c_float, c_float, c_float, c_int, P]),
@@ -134,10 +134,10 @@ SIGNATURES = {
     "vb_qkv_rotary_append": (c_int, [P, c_int, c_int, c_int, c_int, P, c_int, P, P, P, P, P, P, P, c_int, c_int, c_int,
                                      c_int, c_int, c_int, c_int, P, P, c_int, P]),
     "vb_window_attn": (c_int, [P, P, P, P, P, c_int, P, P, P, P, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_float,
-                               c_int, P, C.c_longlong, P, c_int, c_int, c_int, c_int, c_int, c_int, P]),
+                               c_int, P, C.c_longlong, P, c_int, c_int, c_int, c_int, c_int, c_int, P, P]),
     "vb_window_attn_tile_rows": (c_int, []),
     "vb_window_attn_tiled": (c_int, [P, P, P, P, P, c_int, P, P, P, P, P, P, c_int, c_int, c_int, c_int, c_int, c_int,
-                                     c_int, c_int, c_float, c_int, c_int, c_int, c_int, c_int, c_int, P]),
+                                     c_int, c_int, c_float, c_int, c_int, c_int, c_int, c_int, c_int, P, P]),
     "vb_decay_attn": (c_int, [P, P, P, c_int, c_int, c_int, c_int, P, P, P, P, c_int, c_int, c_int, c_int, c_int, c_int,
                               P]),
     "vb_decay_attn_tile_rows": (c_int, [c_int, c_int]),
@@ -159,6 +159,7 @@ SIGNATURES = {
     "vb_linear_batched_gated": (c_int, [P, P, P, c_int, c_int, c_int, c_int, c_int, C.c_longlong, C.c_longlong, C.c_longlong,
                                         c_int, c_int, c_int, c_int, c_float, P, c_int, c_int, P]),
     "vb_pair_hash_rows": (c_int, [P, P, P, P, P, P, P, c_int, c_int, C.c_longlong, C.c_longlong, P]),
+    "vb_hyper_mix_norm": (c_int, [P, c_int, P, P, P, P, P, P, P, P, P, c_int, c_int, c_float, P, c_int, P, P, P, c_int, c_int, P]),
     "vb_short_conv": (c_int, [P, c_int, P, c_int, P, c_int, P, P, P, P, P, P, P, c_int, c_int, c_int, c_int, c_int, c_int, c_int,
                               P]),
     "vb_cast_rows": (c_int, [P, P, c_int, c_int, c_int, c_int, P]),

@@ -33,7 +33,8 @@ constexpr int GEMM_EPI_THREADS = 128;
 enum GemmMode {
   GM_BF16 = 0,      // Y bf16 [T][ldy]
   GM_PARTIAL = 1,   // Y fp32 [split][T][ldy]
-  GM_SILU = 2,      // tile = h gate rows then the h matching up rows; Y bf16 [T][ldy] = silu(gate) * up
+  GM_SILU = 2,      // tile = h gate rows then the h matching up rows; Y bf16 [T][ldy] = silu(gate) * up, or with an
+                    // activation (GemmAct) act(gate) * up in fp32, rounded once
   GM_RESID = 3,     // split-K reduce -> bf16 -> + residual -> bf16 hidden [T][N]; per-tile sums of squares
   GM_ROPE = 4,      // split-K reduce -> bf16 -> RoPE (q, k heads) -> q out / K,V scatter into the page
 };
@@ -363,6 +364,8 @@ __global__ void __launch_bounds__(GEMM_THREADS, 2) gemm_bf16_kernel(const GemmPa
             const float g = fminf(hi ? other : mine, p.glu_limit);
             const float up = fminf(fmaxf(hi ? mine : other, -p.glu_limit), p.glu_limit);
             o[i] = g / (1.0f + expf(-p.glu_slope * g)) * (up + 1.0f);
+          } else if (p.act != GA_NONE) {
+            o[i] = gemm_act(hi ? other : mine, p.act) * (hi ? mine : other);
           } else {
             const float g = round_bf16(hi ? other : mine);
             const float up = round_bf16(hi ? mine : other);
@@ -721,7 +724,7 @@ int vb_gemm_bf16(void* d_y, const void* d_w_tiles, const void* x_map, const void
                  int ldy, int mode, int split_k, int tile_rows, int n_out, int y_tiled, const void* d_bias, int act,
                  void* stream) {
   VB_CHECK_ARG(d_y && d_w_tiles && (x_map || d_x_tiles), "vb_gemm_bf16: null pointer");
-  VB_CHECK_ARG(act >= 0 && act <= 3 && (act == 0 || mode == 0), "vb_gemm_bf16: activation %d is a mode 0 option", act);
+  VB_CHECK_ARG(act >= 0 && act <= 3 && (act == 0 || mode == 0 || mode == 2), "vb_gemm_bf16: activation %d is a mode 0 / 2 option", act);
   VB_CHECK_ARG(!d_bias || mode == 0, "vb_gemm_bf16: bias is a mode 0 option");
   VB_CHECK_ARG(!y_tiled || mode == 2, "vb_gemm_bf16: tiled output is a mode 2 option");
   VB_CHECK_ARG(mode >= 0 && mode <= 2, "vb_gemm_bf16: mode %d", mode);

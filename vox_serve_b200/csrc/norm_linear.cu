@@ -511,7 +511,7 @@ __global__ void postnorm_residual_kernel(float* __restrict__ x, const float* __r
 //   batched: blockIdx.z = g, every group has the rows [0, T): X, Y advance by x_group_stride, o_group_stride elements per
 //            group (heads of one row side by side), gate: Y[r][n] *= sigmoid(gate[r * ld_gate + g])
 // epilogue 0: store (OT);  1: W holds N "gate" rows followed by N "up" rows, store silu(gate) * up (OT);
-//          2: relu(y)^2;  3: gelu(y), exact;  4: gelu(y), tanh form
+//          2: relu(y)^2;  3: gelu(y), exact;  4: gelu(y), tanh form;  5: like 1 with gelu(gate) (tanh form) * up
 // Tile 64 x 64, BK 16, 256 threads, 4 x 4 outputs per thread.
 // ------------------------------------------------------------------------------------------------------------------
 constexpr int LB_M = 64, LB_N = 64, LB_K = 16;
@@ -611,6 +611,8 @@ __global__ void __launch_bounds__(256) linear_kernel(LinearParams p) {
           g = fminf(g, p.glu_limit);
           u = fminf(fmaxf(u, -p.glu_limit), p.glu_limit);
           v = g / (1.f + expf(-p.glu_slope * g)) * (u + 1.f);
+        } else if (p.epi == 5) {
+          v = act_apply(g, 4) * u;
         } else {
           v = g / (1.f + expf(-g)) * u;
         }
@@ -693,7 +695,7 @@ __global__ void __launch_bounds__(128) linear_batched_mma_kernel(LinearParams p)
 template <typename XT, typename WT, typename OT>
 static int launch_linear(const LinearParams& p, int groups, int max_rows, cudaStream_t stream) {
   dim3 grid((max_rows + LB_M - 1) / LB_M, (p.N + LB_N - 1) / LB_N, groups);
-  if (p.epi == 1) VB_LAUNCH_PDL((linear_kernel<XT, WT, OT, 1>), grid, 256, 0, stream, p);
+  if (p.epi == 1 || p.epi == 5) VB_LAUNCH_PDL((linear_kernel<XT, WT, OT, 1>), grid, 256, 0, stream, p);
   else VB_LAUNCH_PDL((linear_kernel<XT, WT, OT, 0>), grid, 256, 0, stream, p);
   return 0;
 }
@@ -912,7 +914,7 @@ int vb_linear(void* d_out, const void* d_x, const void* d_w, int T, int N, int K
               int out_dtype, int epilogue, float alpha, const int32_t* d_row_off, const int32_t* d_gather, int groups,
               long long w_group_stride, float glu_limit, float glu_slope, void* stream) {
   VB_CHECK_ARG(d_out && d_x && d_w && N > 0 && K > 0 && ldx >= K && ldo >= N, "vb_linear: bad arguments");
-  VB_CHECK_ARG(epilogue >= 0 && epilogue <= 4, "vb_linear: epilogue %d", epilogue);
+  VB_CHECK_ARG(epilogue >= 0 && epilogue <= 5, "vb_linear: epilogue %d", epilogue);
   VB_CHECK_ARG(groups >= 1 && (groups == 1 || d_row_off), "vb_linear: grouped launches need row offsets");
   if (T <= 0) return 0;
   LinearParams p{d_out, d_x, d_w, d_row_off, d_gather, T, N, K, ldx, ldo, epilogue, w_group_stride, alpha, 0, 0, nullptr, 0, 0,

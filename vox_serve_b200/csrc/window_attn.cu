@@ -13,12 +13,12 @@
 //                        shared memory and reused by all rows of the tile: mma.sync tensor-core tiles for bf16 heads whose
 //                        sizes are multiples of 16 (keys up to 192 dims, values up to 128), fp32 FMAs otherwise (and always
 //                        in fp32 mode).
-//   vb_qkv_norm_rotary_append, vb_latent_rope_append, vb_head_pair_combine: projection tails with per-head RMS norms, rotation
-//                        in (2i, 2i + 1) or (i, i + half) pairs, a shared rotated key part behind a latent, and the
-//                        combination of two score maps per head.
+//   vb_qkv_norm_rotary_append, vb_latent_rope_append, vb_head_pair_combine: projection tails with projection biases, per-head
+//                        RMS norms of queries, keys and values, rotation in (2i, 2i + 1) or (i, i + half) pairs, a factor per
+//                        query head, a shared rotated key part behind a latent, and the combination of two score maps per head.
 // Besides the sliding window the kernels take a chunk mask (a position sees the keys of its own block of positions), per-token
-// strides of the two caches (a value that is a leading slice of the key row), key heads that share a value head, and an fp32
-// output beside bf16 operands.
+// strides of the two caches (a value that is a leading slice of the key row), key heads that share a value head, an fp32
+// output beside bf16 operands, and a sink per head: one more term e^sink in the softmax's denominator, a key without a value.
 // Cache layout per layer: K [pages][page_size][kv_heads][dim], V [pages][page_size][kv_heads][vdim] unless strides say otherwise.
 #include "../../include/vb_api.h"
 #define VB_PDL_FAMILY 1
@@ -116,14 +116,31 @@ struct LatentTailParams {
   const float* wq;        // [q_rank]
   const float* wc;        // [kv_rank]
   void* cq_out;           // [T][q_rank]
-  void* c_cache;          // [pages][page_size][kv_rank]
+  void* c_cache;          // [pages][page_size][kv_rank + rot]
   const int32_t* row_req;
   const int32_t* pos;
   const int32_t* page_indptr;
   const int32_t* page_indices;
   int page_size;
   float eps;
+  int rot;                // a shared key part of `rot` dims behind the latent's columns, rotated and appended behind it
+  const float* cs;        // [T][2][half] or nullptr (no rotation)
+  int half, layout;
 };
+
+__device__ __forceinline__ float rotated_value(const float* __restrict__ src, const float* __restrict__ w, float r,
+                                               const float* __restrict__ cs, int half, int layout, int d) {
+  // value d of a head after norm (scale r, weight w) and rotation
+  const float x = src[d] * r * (w ? w[d] : 1.f);
+  if (cs == nullptr || d >= 2 * half) return x;
+  int i, partner;
+  bool first;
+  if (layout == 0) { i = d >> 1; first = (d & 1) == 0; partner = d ^ 1; }
+  else { first = d < half; i = first ? d : d - half; partner = first ? d + half : d - half; }
+  const float y = src[partner] * r * (w ? w[partner] : 1.f);
+  const float c = cs[i], sn = cs[half + i];
+  return first ? x * c - y * sn : x * c + y * sn;
+}
 
 template <typename CT>
 __global__ void __launch_bounds__(128) latent_norm_append_kernel(LatentTailParams p) {
@@ -150,14 +167,18 @@ __global__ void __launch_bounds__(128) latent_norm_append_kernel(LatentTailParam
   const float rc = 1.f / sqrtf(sc / p.kv_rank + p.eps);
   const int b = p.row_req[t], ps = p.pos[t];
   const size_t tok = static_cast<size_t>(p.page_indices[p.page_indptr[b] + ps / p.page_size]) * p.page_size + ps % p.page_size;
-  CT* co = static_cast<CT*>(p.c_cache) + tok * p.kv_rank;
+  CT* co = static_cast<CT*>(p.c_cache) + tok * (p.kv_rank + p.rot);
   for (int i = threadIdx.x; i < p.kv_rank; i += 128) co[i] = wa_from_f<CT>(c[i] * rc * p.wc[i]);
+  const float* cs = p.cs ? p.cs + t * 2 * p.half : nullptr;
+  for (int i = threadIdx.x; i < p.rot; i += 128)
+    co[p.kv_rank + i] = wa_from_f<CT>(rotated_value(c + p.kv_rank, nullptr, 1.f, cs, p.half, p.layout, i));
 }
 
 // The tail of a fused q|k|v|.. projection for heads that are normed before they are rotated: every query and key head
 // (for attention with several score maps per head, every map is a head here) is RMS-normed over its dim values with a
 // weight shared by all heads (optional), then its first 2 * half dims are rotated -- pairs (2i, 2i + 1) in the
-// interleaved layout, pairs (i, i + half) in the half layout -- and written out / appended; values are appended as they are.
+// interleaved layout, pairs (i, i + half) in the half layout -- and written out / appended; values are appended as they are,
+// or divided by the root mean square of their head.  A bias per projection column enters first; a factor per query head last.
 // The key cache holds Gk heads per token, the value cache Gv (Gk / Gv key heads read one value head).  One warp per head.
 struct QkvNormTailParams {
   const float* proj;      // [T][ldp]
@@ -176,35 +197,32 @@ struct QkvNormTailParams {
   const int32_t* page_indices;
   int page_size, Hq, Gk, Gv, dim, vdim;
   int stage_lo, stage_hi; // columns of the row staged in shared memory (stage_hi == 0: read from global memory)
+  const float* bias;      // indexed like the row's columns, added to the staged columns; or nullptr
+  const float* q_scale;   // [Hq] or nullptr
+  int v_norm;             // every value head divided by its root mean square over vdim
 };
 
 // Copies floats [lo, hi) of a projection row into shared memory with every load in flight at once (16-byte loads when the
 // row slice is aligned) and returns a pointer that is indexed like the row itself.  The tails below read a row's values
 // more than once (norm, rotation partner) and from many threads: one pass over DRAM, the rest from shared memory.
-__device__ __forceinline__ const float* stage_row(const float* __restrict__ row, int lo, int hi, float* __restrict__ sm) {
+__device__ __forceinline__ const float* stage_row(const float* __restrict__ row, int lo, int hi, float* __restrict__ sm,
+                                                  const float* __restrict__ bias = nullptr) {
   const int n = hi - lo;
-  if (((reinterpret_cast<uintptr_t>(row + lo) & 15) == 0) && (n & 3) == 0) {
-    for (int i = threadIdx.x * 4; i < n; i += blockDim.x * 4)
-      *reinterpret_cast<float4*>(sm + i) = *reinterpret_cast<const float4*>(row + lo + i);
+  if (((reinterpret_cast<uintptr_t>(row + lo) & 15) == 0) && (n & 3) == 0 &&
+      (bias == nullptr || (reinterpret_cast<uintptr_t>(bias + lo) & 15) == 0)) {
+    for (int i = threadIdx.x * 4; i < n; i += blockDim.x * 4) {
+      float4 v = *reinterpret_cast<const float4*>(row + lo + i);
+      if (bias) {
+        const float4 b = *reinterpret_cast<const float4*>(bias + lo + i);
+        v.x += b.x; v.y += b.y; v.z += b.z; v.w += b.w;
+      }
+      *reinterpret_cast<float4*>(sm + i) = v;
+    }
   } else {
-    for (int i = threadIdx.x; i < n; i += blockDim.x) sm[i] = row[lo + i];
+    for (int i = threadIdx.x; i < n; i += blockDim.x) sm[i] = row[lo + i] + (bias ? bias[lo + i] : 0.f);
   }
   __syncthreads();
   return sm - lo;
-}
-
-__device__ __forceinline__ float rotated_value(const float* __restrict__ src, const float* __restrict__ w, float r,
-                                               const float* __restrict__ cs, int half, int layout, int d) {
-  // value d of a head after norm (scale r, weight w) and rotation
-  const float x = src[d] * r * (w ? w[d] : 1.f);
-  if (cs == nullptr || d >= 2 * half) return x;
-  int i, partner;
-  bool first;
-  if (layout == 0) { i = d >> 1; first = (d & 1) == 0; partner = d ^ 1; }
-  else { first = d < half; i = first ? d : d - half; partner = first ? d + half : d - half; }
-  const float y = src[partner] * r * (w ? w[partner] : 1.f);
-  const float c = cs[i], sn = cs[half + i];
-  return first ? x * c - y * sn : x * c + y * sn;
 }
 
 template <typename CT>
@@ -213,7 +231,7 @@ __global__ void __launch_bounds__(256) qkv_norm_rotary_append_kernel(QkvNormTail
   pdl_sync();
   const int t = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const float* row = p.proj + static_cast<size_t>(t) * p.ldp;
-  if (p.stage_hi > 0) row = stage_row(row, p.stage_lo, p.stage_hi, tail_sm);
+  if (p.stage_hi > 0) row = stage_row(row, p.stage_lo, p.stage_hi, tail_sm, p.bias);
   const int b = p.row_req[t], ps = p.pos[t];
   const size_t tok = static_cast<size_t>(p.page_indices[p.page_indptr[b] + ps / p.page_size]) * p.page_size + ps % p.page_size;
   const float* cs = p.cs ? p.cs + static_cast<size_t>(t) * 2 * p.half : nullptr;
@@ -232,7 +250,18 @@ __global__ void __launch_bounds__(256) qkv_norm_rotary_append_kernel(QkvNormTail
       r = 1.f / sqrtf(warp_sum(ss) / p.dim + p.eps);
     }
     CT* dst = (is_q ? q_out : k_out) + h * p.dim;
-    for (int d = lane; d < p.dim; d += 32) dst[d] = wa_from_f<CT>(rotated_value(src, w, r, cs, p.half, p.layout, d));
+    const float mul = is_q && p.q_scale ? p.q_scale[h] : 1.f;
+    for (int d = lane; d < p.dim; d += 32) dst[d] = wa_from_f<CT>(rotated_value(src, w, r, cs, p.half, p.layout, d) * mul);
+  }
+  if (p.v_norm) {
+    for (int h = warp; h < p.Gv; h += 8) {
+      const float* src = row + p.v_off + h * p.vdim;
+      float ss = 0.f;
+      for (int d = lane; d < p.vdim; d += 32) ss = fmaf(src[d], src[d], ss);
+      const float r = 1.f / sqrtf(warp_sum(ss) / p.vdim + p.eps);
+      for (int d = lane; d < p.vdim; d += 32) v_out[h * p.vdim + d] = wa_from_f<CT>(src[d] * r);
+    }
+    return;
   }
   for (int i = threadIdx.x; i < p.Gv * p.vdim; i += 256) v_out[i] = wa_from_f<CT>(row[p.v_off + i]);
 }
@@ -357,7 +386,16 @@ struct WindowAttnParams {
                               // that share a key/value head (grid: served rows x key/value heads x splits)
   int splits;                 // grouped kernel: key tiles are dealt round-robin to `splits` CTAs per (row, key/value head)
   float* part;                // [T][H][splits][vdim + 2]: unnormalised output, running max, running sum of every split
+  const float* sink;          // [H] score of a further key without a value that enters every row's denominator, or nullptr
 };
+
+// what a row's accumulated values are multiplied by, from its running maximum and sum: 1 / l, or with a sink
+// e^(m - M) / (l e^(m - M) + e^(sink - M)), M = max(m, sink)
+__device__ __forceinline__ float wa_inv(const WindowAttnParams& p, int h, float m, float l) {
+  if (p.sink == nullptr) return 1.f / l;
+  const float s = p.sink[h], M = fmaxf(m, s), c = expf(m - M);
+  return c / (l * c + expf(s - M));
+}
 
 // first visible key of a query at position pos: the sliding window's start, the start of the position's chunk, or 0
 __device__ __forceinline__ int wa_first_key(const WindowAttnParams& p, int pos) {
@@ -497,7 +535,7 @@ __global__ void __launch_bounds__(WA_WARPS * 32) window_attn_kernel(WindowAttnPa
       }
     }
   }
-  const float inv = 1.f / l;
+  const float inv = wa_inv(p, h, m, l);
   const size_t out0 = static_cast<size_t>(t) * p.H * p.vdim + h * p.vdim;
   const float* gate = p.gate ? p.gate + static_cast<size_t>(t) * p.ld_gate + h * p.vdim : nullptr;
 #pragma unroll
@@ -604,7 +642,7 @@ __global__ void __launch_bounds__(256) window_attn_tiled_kernel(WindowAttnParams
   }
   if (!row_ok) return;
   const int t = row0 + r;
-  const float inv = 1.f / l;
+  const float inv = wa_inv(p, h, m, l);
   const size_t out0 = static_cast<size_t>(t) * p.H * dv + h * dv;
   const float* gate = p.gate ? p.gate + static_cast<size_t>(t) * p.ld_gate + h * dv : nullptr;
 #pragma unroll
@@ -710,7 +748,7 @@ __global__ void __launch_bounds__(128) window_attn_group_kernel(WindowAttnParams
       }
       continue;
     }
-    const float inv = 1.f / l[u];
+    const float inv = wa_inv(p, h, m[u], l[u]);
     const size_t out0 = static_cast<size_t>(t) * p.H * dv + h * dv;
     const float* gate = p.gate ? p.gate + static_cast<size_t>(t) * p.ld_gate + h * dv : nullptr;
 #pragma unroll
@@ -736,9 +774,10 @@ __global__ void __launch_bounds__(64) window_attn_merge_kernel(WindowAttnParams 
   if (threadIdx.x < 32) {
     const int s = threadIdx.x;
     const float m = s < S ? pt[s * (dv + 2) + dv] : -INFINITY, l = s < S ? pt[s * (dv + 2) + dv + 1] : 0.f;
-    const float M = warp_max(m);
+    float M = warp_max(m);
+    if (p.sink) M = fmaxf(M, p.sink[h]);
     const float w = m == -INFINITY ? 0.f : expf(m - M);
-    const float L = warp_sum(l * w);
+    const float L = warp_sum(l * w) + (p.sink ? expf(p.sink[h] - M) : 0.f);
     wgt[s] = w / L;
   }
   __syncthreads();
@@ -956,7 +995,8 @@ __global__ void __launch_bounds__(128) window_attn_mma_kernel(WindowAttnParams p
     }
     return;
   }
-  const float iA = okA ? 1.f / lA : 0.f, iB = okB ? 1.f / lB : 0.f;
+  const float iA = okA ? wa_inv(p, p.row_heads ? g * nrows + rA : h, mA, lA) : 0.f;
+  const float iB = okB ? wa_inv(p, p.row_heads ? g * nrows + rB : h, mB, lB) : 0.f;
   __nv_bfloat16* out = static_cast<__nv_bfloat16*>(p.out);
 #pragma unroll
   for (int n = 0; n < F_NT; ++n) {
@@ -999,7 +1039,8 @@ int vb_qkv_norm_rotary_append(const float* d_proj, int ldp, int q_off, int k_off
                               int layout, const float* d_q_norm, const float* d_k_norm, float eps, void* d_q_out,
                               void* d_k_cache, void* d_v_cache, const int32_t* d_row_req, const int32_t* d_pos,
                               const int32_t* d_page_indptr, const int32_t* d_page_indices, int page_size, int T, int Hq, int Gk,
-                              int Gv, int dim, int vdim, int dtype, void* stream) {
+                              int Gv, int dim, int vdim, int dtype, const float* d_bias, const float* d_q_scale, int v_norm,
+                              void* stream) {
   VB_CHECK_ARG(d_proj && d_q_out && d_k_cache && d_v_cache && d_row_req && d_pos && d_page_indptr && d_page_indices,
                "vb_qkv_norm_rotary_append: null pointer");
   VB_CHECK_ARG(Hq > 0 && Gk > 0 && Gv > 0 && dim > 0 && vdim > 0 && page_size > 0 && half >= 0 && 2 * half <= dim &&
@@ -1008,7 +1049,7 @@ int vb_qkv_norm_rotary_append(const float* d_proj, int ldp, int q_off, int k_off
   if (T <= 0) return 0;
   QkvNormTailParams p{d_proj, ldp, q_off, k_off, v_off, half > 0 ? d_cs : nullptr, half, layout, d_q_norm, d_k_norm, eps,
                       d_q_out, d_k_cache, d_v_cache, d_row_req, d_pos, d_page_indptr, d_page_indices, page_size, Hq, Gk, Gv,
-                      dim, vdim, 0, 0};
+                      dim, vdim, 0, 0, d_bias, d_q_scale, v_norm};
   // the q | k | v columns of a row are staged in shared memory when they lie side by side and fit
   const int lo = min(q_off, min(k_off, v_off)), hi = max(q_off + Hq * dim, max(k_off + Gk * dim, v_off + Gv * vdim));
   size_t smem = 0;
@@ -1016,6 +1057,7 @@ int vb_qkv_norm_rotary_append(const float* d_proj, int ldp, int q_off, int k_off
     p.stage_lo = lo; p.stage_hi = hi;
     smem = static_cast<size_t>(hi - lo) * sizeof(float);
   }
+  VB_CHECK_ARG(!d_bias || p.stage_hi > 0, "vb_qkv_norm_rotary_append: a bias needs q, k, v columns side by side that fit shared memory");
   if (dtype == 1) {
     if (smem > 48 * 1024) VB_CHECK_CUDA(cudaFuncSetAttribute(qkv_norm_rotary_append_kernel<float>, cudaFuncAttributeMaxDynamicSharedMemorySize, VB_MAX_DYN_SMEM));
     VB_LAUNCH_PDL(qkv_norm_rotary_append_kernel<float>, T, 256, smem, stream, p);
@@ -1093,14 +1135,15 @@ int vb_qkv_rotary_append(const float* d_proj, int ldp, int q_off, int k_off, int
 int vb_latent_norm_append(const float* d_proj, int ldp, int q_off, int c_off, int q_rank, int kv_rank, const float* d_wq,
                           const float* d_wc, void* d_cq_out, void* d_c_cache, const int32_t* d_row_req, const int32_t* d_pos,
                           const int32_t* d_page_indptr, const int32_t* d_page_indices, int page_size, int T, float eps,
-                          int dtype, void* stream) {
+                          int rot, const float* d_cs, int half, int layout, int dtype, void* stream) {
   VB_CHECK_ARG(d_proj && d_wq && d_cq_out && q_rank > 0 && q_off >= 0 && q_off + q_rank <= ldp,
                "vb_latent_norm_append: bad query latent");
   VB_CHECK_ARG(!d_c_cache || (d_wc && d_row_req && d_pos && d_page_indptr && d_page_indices && kv_rank > 0 && page_size > 0 &&
-                              c_off >= 0 && c_off + kv_rank <= ldp), "vb_latent_norm_append: bad key/value latent");
+                              rot >= 0 && 2 * half <= rot && half >= 0 && (layout == 0 || layout == 1) &&
+                              c_off >= 0 && c_off + kv_rank + rot <= ldp), "vb_latent_norm_append: bad key/value latent");
   if (T <= 0) return 0;
   LatentTailParams p{d_proj, ldp, q_off, c_off, q_rank, kv_rank, d_wq, d_wc, d_cq_out, d_c_cache, d_row_req, d_pos,
-                     d_page_indptr, d_page_indices, page_size, eps};
+                     d_page_indptr, d_page_indices, page_size, eps, rot, half > 0 ? d_cs : nullptr, half, layout};
   if (dtype == 1) VB_LAUNCH_PDL(latent_norm_append_kernel<float>, T, 128, 0, stream, p);
   else VB_LAUNCH_PDL(latent_norm_append_kernel<bf16>, T, 128, 0, stream, p);
   return 0;
@@ -1110,7 +1153,7 @@ int vb_window_attn(void* d_out, const void* d_q, const void* d_k_cache, const vo
                    int ld_gate, const int32_t* d_row_req, const int32_t* d_pos, const int32_t* d_page_indptr,
                    const int32_t* d_page_indices, int T, int H, int G, int dim, int vdim, int page_size, int window,
                    float scale, int dtype, float* d_part, long long part_floats, const int32_t* d_row_list, int head_rows,
-                   int chunk, int k_ld, int v_ld, int v_share, int out_f32, void* stream) {
+                   int chunk, int k_ld, int v_ld, int v_share, int out_f32, const float* d_sink, void* stream) {
   VB_CHECK_ARG(d_out && d_q && d_k_cache && d_v_cache && d_row_req && d_pos && d_page_indptr && d_page_indices,
                "vb_window_attn: null pointer");
   VB_CHECK_ARG(H > 0 && G > 0 && H % G == 0 && dim > 0 && vdim > 0 && vdim <= 32 * WA_MAXU && page_size > 0,
@@ -1122,7 +1165,7 @@ int vb_window_attn(void* d_out, const void* d_q, const void* d_k_cache, const vo
   if (v_ld <= 0) v_ld = (G / v_share) * vdim;
   WindowAttnParams p{d_q, d_k_cache, d_v_cache, d_out, d_gate, ld_gate, d_row_req, d_pos, d_page_indptr, d_page_indices,
                      nullptr, nullptr, nullptr, T, H, G, dim, vdim, page_size, window, chunk, k_ld, v_ld, v_share, out_f32,
-                     scale, d_row_list, 0, 1, d_part};
+                     scale, d_row_list, 0, 1, d_part, d_sink};
   const int R = H / G;
   const bool mma_ok = dtype == 0 && dim % 16 == 0 && vdim % 16 == 0 && dim <= 16 * F_KB && vdim <= 8 * F_NT &&
                       k_ld % 8 == 0 && v_ld % 8 == 0;
@@ -1186,7 +1229,7 @@ int vb_window_attn_tiled(void* d_out, const void* d_q, const void* d_k_cache, co
                          int ld_gate, const int32_t* d_pos, const int32_t* d_page_indptr, const int32_t* d_page_indices,
                          const int32_t* d_qo_indptr, const int32_t* d_tile_req, const int32_t* d_tile_row0, int n_tiles,
                          int T, int H, int G, int dim, int vdim, int page_size, int window, float scale, int dtype,
-                         int chunk, int k_ld, int v_ld, int v_share, int out_f32, void* stream) {
+                         int chunk, int k_ld, int v_ld, int v_share, int out_f32, const float* d_sink, void* stream) {
   VB_CHECK_ARG(d_out && d_q && d_k_cache && d_v_cache && d_pos && d_page_indptr && d_page_indices && d_qo_indptr &&
                d_tile_req && d_tile_row0, "vb_window_attn_tiled: null pointer");
   VB_CHECK_ARG(H > 0 && G > 0 && H % G == 0 && dim > 0 && vdim > 0 && vdim <= 4 * WT_MAXD && page_size > 0,
@@ -1198,7 +1241,7 @@ int vb_window_attn_tiled(void* d_out, const void* d_q, const void* d_k_cache, co
   if (v_ld <= 0) v_ld = (G / v_share) * vdim;
   WindowAttnParams p{d_q, d_k_cache, d_v_cache, d_out, d_gate, ld_gate, nullptr, d_pos, d_page_indptr, d_page_indices,
                      d_qo_indptr, d_tile_req, d_tile_row0, T, H, G, dim, vdim, page_size, window, chunk, k_ld, v_ld, v_share,
-                     out_f32, scale, nullptr, 0, 1, nullptr};
+                     out_f32, scale, nullptr, 0, 1, nullptr, d_sink};
   dim3 grid(n_tiles, H);
   if (dtype == 0 && dim % 16 == 0 && vdim % 16 == 0 && dim <= 16 * F_KB && vdim <= 8 * F_NT && k_ld % 8 == 0 && v_ld % 8 == 0) {
     const size_t msmem = 2 * static_cast<size_t>(FN) * (dim + 8 + vdim + 8) * sizeof(__nv_bfloat16);      // two stages

@@ -24,7 +24,11 @@ feed-forward (``_forward_gated``).  A fourth, ``post`` (what a sublayer returns 
 itself -- the mixer through a short causal input convolution with state), carries latent attention in a window with a gate per
 output value and rows that layers may share, and a pair of mixers side by side -- attention whose weights are sigmoids over a
 window plus pooled blocks, and a selective scan -- with a group-limited softmax router over clamped gated experts, a hashed
-token-pair embedding and a tied head (``_forward_post`` at the end of this file).
+token-pair embedding and a tied head (``_forward_post``).  A fifth, ``hyper`` (hyper-connections: the stream is several
+copies; a sublayer reads a weighted sum of them through a norm and an input convolution with state, and its output enters all of
+them beside a mix of the old ones), carries latent attention with a query latent and a rotated part, and grouped-head attention
+with projection biases, values of unit RMS, a factor per head on the scores and a sink in the softmax's denominator
+(``_forward_hyper`` at the end of this file).
 
 Precision: ``dtype`` bfloat16 keeps projections' operands, q / k / v, the page cache and the attention output in bf16 with
 fp32 accumulation; norms, softmax, router, residual, recurrent state, decays and the lightning path after its projection
@@ -57,7 +61,7 @@ class RotaryConfig:
     original: float = 8192.0
     layout: str = "interleaved"          # "interleaved": dim 2i goes with 2i + 1; "half": dim i goes with i + dims / 2
     scaling: str = "wavelength"          # "wavelength" (Llama-3.1 style, low / high) | "yarn" (fast / slow turns, ramp over the
-    #                                      pair index, cos and sin times 0.1 ln(factor) + 1)
+    #                                      pair index, cos and sin times 0.1 ln(factor) + 1) | "linear" (every frequency / factor)
     fast: float = 32.0
     slow: float = 1.0
 
@@ -71,7 +75,7 @@ class RotaryConfig:
     def frequencies(self) -> torch.Tensor:
         """float64 [dims / 2]: base^(-2i/dims).  "wavelength" scaling: wavelengths above original/low are slowed by
         ``factor``, those below original/high kept, the band in between interpolated linearly in original/wavelength.
-        "yarn" scaling: with d(t) = dims ln(original / (2 pi t)) / (2 ln base) the pair index that turns t times within
+        "linear" scaling: every frequency divided by ``factor``.  "yarn" scaling: with d(t) = dims ln(original / (2 pi t)) / (2 ln base) the pair index that turns t times within
         ``original`` positions, pairs up to lo = max(floor d(fast), 0) keep their frequency, pairs from
         hi = min(ceil d(slow), dims - 1) on are slowed by ``factor``, linearly mixed in between."""
         if self.factor is not None and self.scaling == "yarn":
@@ -87,7 +91,9 @@ class RotaryConfig:
         out = []
         for i in range(self.dims // 2):
             f = self.base ** (-2.0 * i / self.dims)
-            if self.factor is not None:
+            if self.factor is not None and self.scaling == "linear":
+                f = f / self.factor
+            elif self.factor is not None:
                 wl = 2.0 * math.pi / f
                 if wl < self.original / self.high:
                     pass
@@ -111,6 +117,10 @@ class WindowAttentionConfig:
     rotary: Optional[RotaryConfig] = None
     v_mix: bool = False
     gate: bool = True
+    bias: bool = False                    # biases on the q, k, v and output projections
+    value_norm: bool = False              # every value head divided by its root mean square over vdim (cached so)
+    head_factor: bool = False             # scores times one number per query head
+    sink: Optional[float] = None          # score of a further key without a value in every softmax (0: one joins the denominator)
 
 
 @dataclass
@@ -225,10 +235,12 @@ class DenseMLPConfig:
 
 @dataclass
 class GluMLPConfig:
-    """down(g * sigmoid(slope * g) * (u + 1)) with g = min(gate h, limit), u = clamp(up h, -limit, limit)."""
+    """act "clamped": down(g * sigmoid(slope * g) * (u + 1)) with g = min(gate h, limit), u = clamp(up h, -limit, limit).
+    act "gelu_tanh": down(gelu(gate h) * up h), the tanh form of gelu."""
     ff: int
-    limit: float
+    limit: float = 0.0
     slope: float = 1.702
+    act: str = "clamped"
 
 
 @dataclass
@@ -269,6 +281,8 @@ class HybridConfig:
     #                                       "gated": pre-norm, x += sigmoid(W_r h + b) * sublayer(h) with h = norm(x), mixer then ff
     #                                       "post": x += norm(sublayer(x)): only what a sublayer returns is normed; the sublayers
     #                                       read the stream itself (the mixer through the input convolution, if any)
+    #                                       "hyper": the stream is ``streams`` copies; u = sum_s in[s] x_s, y = sublayer(c(norm(u))),
+    #                                       x_t <- sum_s mix[s, t] x_s + out[t] y, mixer then ff, c the input convolution
     norm: str = "layernorm"               # "layernorm" (weight and bias) | "rmsnorm" (weight) | "rmsnorm_scalar" (one number) |
     #                                       "rmsnorm_offset" (the stored weight is an offset from one: x / rms * (1 + w))
     residual_mult: float = 1.0            # m of the parallel form
@@ -277,14 +291,15 @@ class HybridConfig:
     logit_softcap: float = 0.0            # logits <- cap * tanh(logits / cap) (0: none)
     embed_scale: float = 1.0              # the embedding rows are multiplied by this
     # layers loop_start .. loop_stop - 1 run loop_times times in a row with the same weights; every pass has its own cache and
-    # state, and before each pass but the first the embedding output is added to the stream
+    # state, and ("gated" blocks) before each pass but the first the embedding output is added to the stream
     loop_start: int = 0
     loop_stop: int = 0
     loop_times: int = 1
     tied_head: bool = False               # the output head is the embedding table itself (unscaled); no "head" tensor
     pair_embed: Optional[PairEmbedConfig] = None   # a hashed (previous token, token) embedding added to the token's
-    input_conv: int = 0                   # "post" blocks: the mixer reads h + conv(h), a causal convolution of this many taps
-    #                                       over time on every channel of the stream (0: it reads h)
+    input_conv: int = 0                   # "post" blocks: the mixer, "hyper" blocks: both sublayers read h + conv(h), a causal
+    #                                       convolution of this many taps over time on every channel of what they read (0: h)
+    streams: int = 1                      # copies of the residual stream ("hyper" blocks; at the end they are summed)
 
     def runs(self) -> List[Tuple[int, bool]]:
         """(layer index, does a repeated pass start here) for every layer run in order.  Caches and states are kept per run."""
@@ -419,6 +434,9 @@ class HybridWeights:
                 continue
             if cfg.block == "post":
                 self.layers.append(self._load_post_layer(sd, p, i, L, norm))
+                continue
+            if cfg.block == "hyper":
+                self.layers.append(self._load_hyper_layer(sd, p, i, L, norm))
                 continue
             if cfg.block == "parallel":
                 w: Dict[str, Any] = {"norm1": vec(p + "norm1")}
@@ -581,6 +599,58 @@ class HybridWeights:
                 raise VoxB200Error(f"layer {i}: router shape does not match the configuration")
         return w
 
+    def _load_hyper_layer(self, sd, p: str, i: int, L: "HybridLayerConfig", norm) -> Dict[str, Any]:
+        """A layer with hyper-connections: per sublayer q (1 mixer, 2 feed-forward) ``l<i>.norm<q>``, ``l<i>.canon<q>`` (input
+        convolution [width, taps]), ``l<i>.hc<q>.{in [S], out [S], mix [S, S] (from, to)}``; ``l<i>.mix.*``,
+        ``l<i>.mlp.{gate,up,down}``.
+          latent attention: as ``_load_latent``, with a rotated part behind every query head and behind the latent
+          attention: q | k | v (| g) as ONE projection; biases ``.{q,k,v}.b`` stacked like its columns, ``.o.b``; ``.temp`` [H]"""
+        mat, vec, dense, cfg, W, m = self._mat, self._vec, self._dense, self.cfg, self.cfg.width, L.mixer
+        S = cfg.streams
+        w: Dict[str, Any] = {}
+        for q in ((1, 2) if L.mlp is not None else (1,)):
+            w[f"norm{q}"] = norm(p + f"norm{q}")[0]
+            w[f"hc{q}"] = tuple(vec(p + f"hc{q}.{n}") for n in ("in", "out", "mix"))
+            if w[f"hc{q}"][0].numel() != S or w[f"hc{q}"][1].numel() != S or tuple(w[f"hc{q}"][2].shape) != (S, S):
+                raise VoxB200Error(f"layer {i}: hyper-connection shapes do not match {S} streams")
+            if cfg.input_conv:
+                w[f"canon{q}"] = vec(p + f"canon{q}")
+                if tuple(w[f"canon{q}"].shape) != (W, cfg.input_conv):
+                    raise VoxB200Error(f"layer {i}: input convolution shape does not match the configuration")
+        if L.kind == "latent":
+            self._load_latent(sd, p, i, m, w)
+        elif L.kind == "attention":
+            nq, nk, nv = m.heads * m.dim, m.kv_heads * m.dim, m.kv_heads * m.vdim
+            w["qkvg"] = mat(*[p + "mix." + n for n in (("q", "k", "v", "g") if m.gate else ("q", "k", "v"))])
+            w["o"] = mat(p + "mix.o")
+            if (tuple(w["qkvg"].shape) != (nq + nk + nv + (m.heads * m.vdim if m.gate else 0), W) or
+                    tuple(sd[p + "mix.q"].shape) != (nq, W) or tuple(sd[p + "mix.k"].shape) != (nk, W) or
+                    tuple(w["o"].shape) != (W, m.heads * m.vdim)):
+                raise VoxB200Error(f"layer {i}: attention shapes do not match the configuration")
+            if m.bias:
+                w["qkv_b"] = torch.cat([vec(p + f"mix.{n}.b") for n in ("q", "k", "v")], 0).contiguous()
+                w["o_b"] = vec(p + "mix.o.b")
+                if w["qkv_b"].numel() != nq + nk + nv or w["o_b"].numel() != W:
+                    raise VoxB200Error(f"layer {i}: attention bias shapes do not match the configuration")
+            if m.head_factor:
+                w["head_factor"] = vec(p + "mix.temp")
+                if w["head_factor"].numel() != m.heads:
+                    raise VoxB200Error(f"layer {i}: one score factor per head")
+            if m.sink is not None:
+                w["sink"] = torch.full((m.heads,), m.sink, dtype=F32, device=self.device)
+            w["qkvg"], w["o"] = dense(w["qkvg"]), dense(w["o"])
+        else:
+            raise VoxB200Error(f"layer {i}: mixer '{L.kind}' is not available in hyper-connected blocks")
+        f = L.mlp
+        if f is not None:
+            if not isinstance(f, GluMLPConfig):
+                raise VoxB200Error(f"layer {i}: hyper-connected blocks take a gated dense feed-forward")
+            if (tuple(sd[p + "mlp.gate"].shape) != (f.ff, W) or tuple(sd[p + "mlp.up"].shape) != (f.ff, W) or
+                    tuple(sd[p + "mlp.down"].shape) != (W, f.ff)):
+                raise VoxB200Error(f"layer {i}: feed-forward shapes do not match the configuration")
+            w["gu"], w["down"] = self._gate_up(p + "mlp.gate", p + "mlp.up"), dense(mat(p + "mlp.down"))
+        return w
+
     def _load_gated_layer(self, sd, p: str, i: int, L: "HybridLayerConfig", norm) -> Dict[str, Any]:
         """A pre-norm layer with gated residuals: ``l<i>.norm1`` / ``norm2``, ``l<i>.rg1[.b]`` / ``rg2[.b]`` (the gates of the
         mixer's and the feed-forward's residual), ``l<i>.mix.*``, ``l<i>.mlp.{gate,up,down}``.  The mixer's gate reads the
@@ -651,7 +721,8 @@ class HybridWeights:
 
     def _load_latent(self, sd, p: str, i: int, m: "LatentAttentionConfig", w: Dict[str, Any]) -> None:
         """``l<i>.mix.{dq, dq.norm, uq, dkv, dkv.norm, uk, uv, g, o}``: dq | dkv | g become one projection (a layer that
-        reads another layer's latents has no dkv); uk is kept per head and transposed ([H, kv_rank, dim]: it carries a
+        reads another layer's latents has no dkv; with a rotated part, dkv has rot_dim rows more and every query head of uq
+        too); uk is kept per head and transposed ([H, kv_rank, dim]: it carries a
         head's query into latent space), uv per head ([H, vdim, kv_rank]: it expands a head's latent-space output)."""
         mat, vec, dense, W = self._mat, self._vec, self._dense, self.cfg.width
         own = m.kv_from is None
@@ -662,10 +733,12 @@ class HybridWeights:
                                    "projects its own latents of the same rank")
         names = [p + "mix.dq"] + ([p + "mix.dkv"] if own else []) + [p + "mix.g"]
         down = mat(*names)
-        if tuple(down.shape) != (m.q_rank + (m.kv_rank if own else 0) + m.heads, W):
+        if m.rot_dim and not own:
+            raise VoxB200Error(f"layer {i}: a query latent with a rotated part needs latents of the layer's own")
+        if tuple(down.shape) != (m.q_rank + (m.kv_rank + m.rot_dim if own else 0) + m.heads, W):
             raise VoxB200Error(f"layer {i}: latent projection shapes do not match the configuration")
         uq, uk, uv, o = mat(p + "mix.uq"), mat(p + "mix.uk"), mat(p + "mix.uv"), mat(p + "mix.o")
-        if (tuple(uq.shape) != (m.heads * m.dim, m.q_rank) or tuple(uk.shape) != (m.heads * m.dim, m.kv_rank) or
+        if (tuple(uq.shape) != (m.heads * (m.dim + m.rot_dim), m.q_rank) or tuple(uk.shape) != (m.heads * m.dim, m.kv_rank) or
                 tuple(uv.shape) != (m.heads * m.vdim, m.kv_rank) or tuple(o.shape) != (W, m.heads * m.vdim)):
             raise VoxB200Error(f"layer {i}: latent attention shapes do not match the configuration")
         w["lat_in"], w["uq"], w["o"] = dense(down), dense(uq), dense(o)
@@ -739,7 +812,7 @@ class HybridCache:
     per linear-attention layer a state [slots, H, dim, vdim] and per minGRU layer a state [slots, width] in fp32; per mixer
     pair K / V pages of its attention, fp32 pooled blocks [pages, ceil(page / pool), G, dim / vdim], the scan's state
     [slots, inner, N] and the last inputs of its short convolutions [slots, taps - 1, channels]; per layer of a stack with an
-    input convolution its last inputs [slots, taps - 1, width]; with a token-pair embedding the last token of every slot.  A layer
+    input convolution its last inputs [slots, taps - 1, width] (hyper-connected blocks: one for each sublayer); with a token-pair embedding the last token of every slot.  A layer
     that a loop runs several times has one of these per pass.  Pages and slots are handed out by the worker; a slot's state is treated as zero by
     the kernels when its request starts at position 0, so nothing is cleared on reuse."""
 
@@ -786,8 +859,10 @@ class HybridCache:
                 self.state[i] = torch.zeros(num_slots, r.inner, r.state, dtype=F32, device=device)
             else:
                 self.state[i] = torch.zeros(num_slots, m.heads, m.dim, m.vdim, dtype=F32, device=device)
-            if cfg.block == "post" and cfg.input_conv > 1:
+            if cfg.block in ("post", "hyper") and cfg.input_conv > 1:
                 self.conv[(i, "in")] = torch.zeros(num_slots, cfg.input_conv - 1, cfg.width, dtype=F32, device=device)
+                if cfg.block == "hyper" and L.mlp is not None:
+                    self.conv[(i, "ff")] = torch.zeros(num_slots, cfg.input_conv - 1, cfg.width, dtype=F32, device=device)
 
     def nbytes(self) -> int:
         seen = {t.data_ptr(): t for d in (self.k, self.v, self.state, self.k_pool, self.v_pool, self.conv)
@@ -883,6 +958,13 @@ class HybridEngine:
             self.pair_rows = torch.zeros(R, dtype=I32, device=dev)
         if cfg.input_conv > 16:
             raise VoxB200Error("input convolution: at most 16 taps")
+        if cfg.block == "hyper":
+            if not 1 <= cfg.streams <= 16:
+                raise VoxB200Error(f"hyper-connections: {cfg.streams} streams (1 to 16)")
+            self.xs = torch.zeros(R, cfg.streams, W, dtype=F32, device=dev)   # the copies of the stream
+            self.h32 = torch.zeros(R, W, dtype=F32, device=dev) if cfg.input_conv else None   # what an input convolution reads
+        if any(m.q_rank and m.rot_dim for m in lat):
+            self.q_up = torch.zeros(R * max(m.heads * (m.dim + m.rot_dim) for m in lat if m.q_rank and m.rot_dim), dtype=F32, device=dev)
         if cfg.block == "gated":
             self.rg = torch.zeros(R, W, dtype=F32, device=dev)         # the feed-forward's residual gate before its sigmoid
             # the embedding output, added again before every repeated pass over the looped layers
@@ -1010,19 +1092,31 @@ class HybridEngine:
     def _latent(self, i: int, m: LatentAttentionConfig, w: Dict[str, Any], s: StepInputs) -> torch.Tensor:
         """Latent attention in its absorbed form: a head's score q . (U_k c) equals (U_k^T q) . c and its output
         U_v (sum_j p_j c_j), so the cached latents serve every head directly as one shared key = value head of kv_rank
-        dims, and neither keys nor values are ever formed per token."""
-        T, H, R = s.T, m.heads, m.kv_rank
+        dims, and neither keys nor values are ever formed per token.  With a rotated part the cached row is [c | k_r] and a
+        head's query [U_k^T q_u | q_r]: the value is the row's leading kv_rank dims."""
+        T, H, R, Rd = s.T, m.heads, m.kv_rank, m.rot_dim
         own = m.kv_from is None
-        P = m.q_rank + (R if own else 0) + H
+        P = m.q_rank + (R + Rd if own else 0) + H
         proj = self._proj(self.h[:T], w["lat_in"], self.proj[:T * P].view(T, P))
         cq = self.cq[:T * m.q_rank].view(T, m.q_rank)
         cache = self.cache.k[i]
+        cs, half = (self.cs[m.rotary.key()], m.rotary.dims // 2) if (m.rotary is not None and Rd) else (None, 0)
+        layout = m.rotary.layout if m.rotary is not None else "half"
         ops.latent_norm_append(proj, 0, m.q_rank, m.q_rank, R, w["dq_norm"], w.get("dkv_norm"), cq, cache if own else None,
-                               s.row_req, s.pos, s.page_indptr, s.page_indices, T, self.cfg.eps)
-        q = self._proj_ct(cq, w["uq"], self.q[:T * H * m.dim].view(T, H * m.dim))
-        q_lat = ops.linear_batched(q.view(T, H, m.dim), w["uk_t"], self.q_lat[:T * H * R].view(T, H, R))
+                               s.row_req, s.pos, s.page_indptr, s.page_indices, T, self.cfg.eps, rot=Rd, cs=cs, half=half,
+                               layout=layout)
+        q_lat = self.q_lat[:T * H * (R + Rd)].view(T, H, R + Rd)
+        if Rd:          # the up-projected queries stay fp32 until their rotated parts are rotated
+            q = self.q[:T * H * m.dim].view(T, H, m.dim)
+            q32 = self._proj(cq, w["uq"], self.q_up[:T * H * (m.dim + Rd)].view(T, H * (m.dim + Rd)))
+            ops.latent_rope_append(q32, 0, 0, H, m.dim, Rd, R, None, cs, half, layout, q, q_lat, None, s.row_req, s.pos,
+                                   s.page_indptr, s.page_indices, T, self.cfg.eps)
+        else:
+            q = self._proj_ct(cq, w["uq"], self.q[:T * H * m.dim].view(T, H * m.dim)).view(T, H, m.dim)
+        ops.linear_batched(q, w["uk_t"], q_lat[:, :, :R])
         o_lat = self.o_lat[:T * H * R].view(T, H * R)
-        self._run_attention(s, q_lat.view(T, H * R), cache, cache, o_lat, None, H, 1, R, R, 0, m.scale, head_rows=True)
+        self._run_attention(s, q_lat.view(T, H * (R + Rd)), cache, cache, o_lat, None, H, 1, R + Rd, R, m.window, m.scale,
+                            head_rows=True, k_ld=R + Rd, v_ld=R + Rd)
         out = self.mix_out[:T * H * m.vdim].view(T, H, m.vdim)
         ops.linear_batched(o_lat.view(T, H, R), w["uv"], out, gate=proj[:, P - H:])
         return self._proj(out.view(T, H * m.vdim), w["o"], self.y[:T])
@@ -1035,20 +1129,25 @@ class HybridEngine:
     def _attention(self, i: int, m: WindowAttentionConfig, w: Dict[str, Any], s: StepInputs) -> torch.Tensor:
         T, W = s.T, self.cfg.width
         nq, nk, nv = m.heads * m.dim, m.kv_heads * m.dim, m.kv_heads * m.vdim
-        P = nq + nk + nv + m.heads * m.vdim
+        P = nq + nk + nv + (m.heads * m.vdim if m.gate else 0)
         proj = self._proj(self.h[:T], w["qkvg"], self.proj[:T * P].view(T, P))
-        cs, half = None, 0
+        cs, half, layout = None, 0, "half"
         if m.rotary is not None:
-            cs, half = self.cs[m.rotary.key()], m.rotary.dims // 2
+            cs, half, layout = self.cs[m.rotary.key()], m.rotary.dims // 2, m.rotary.layout
         q = self.q[:T * nq].view(T, nq)
-        vmix = 0 if not m.v_mix else (1 if i == self.first_vmix else 2)
-        ops.qkv_rotary_append(proj, 0, nq, nq + nk, cs, half, q, self.cache.k[i], self.cache.v[i], s.row_req, s.pos,
-                              s.page_indptr, s.page_indices, T, m.heads, m.kv_heads, m.dim, m.vdim, vmix,
-                              self.v_first if m.v_mix else None, w.get("vmix") if vmix == 2 else None)
+        if m.bias or m.value_norm or m.head_factor or layout == "half":
+            ops.qkv_norm_rotary_append(proj, 0, nq, nq + nk, cs, half, layout, None, None, self.cfg.eps, q, self.cache.k[i],
+                                       self.cache.v[i], s.row_req, s.pos, s.page_indptr, s.page_indices, T, m.heads,
+                                       bias=w.get("qkv_b"), q_scale=w.get("head_factor"), v_norm=m.value_norm)
+        else:
+            vmix = 0 if not m.v_mix else (1 if i == self.first_vmix else 2)
+            ops.qkv_rotary_append(proj, 0, nq, nq + nk, cs, half, q, self.cache.k[i], self.cache.v[i], s.row_req, s.pos,
+                                  s.page_indptr, s.page_indices, T, m.heads, m.kv_heads, m.dim, m.vdim, vmix,
+                                  self.v_first if m.v_mix else None, w.get("vmix") if vmix == 2 else None)
         out = self.mix_out[:T * m.heads * m.vdim].view(T, m.heads * m.vdim)
         gate = proj[:, nq + nk + nv:] if m.gate else None
         self._run_attention(s, q, self.cache.k[i], self.cache.v[i], out, gate, m.heads, m.kv_heads, m.dim, m.vdim, m.window,
-                            m.scale)
+                            m.scale, sink=w.get("sink"))
         return self._proj(out, w["o"], self.y[:T])
 
     def _lightning(self, i: int, m: DecayAttentionConfig, w: Dict[str, Any], s: StepInputs) -> torch.Tensor:
@@ -1196,6 +1295,8 @@ class HybridEngine:
             return self._forward_gated(s)
         if cfg.block == "post":
             return self._forward_post(s)
+        if cfg.block == "hyper":
+            return self._forward_hyper(s)
         x, h, y = self.x[:T], self.h[:T], self.y[:T]
         ops.embed_rows_f32(w.embed, s.ids, x, w.pos, s.pos if w.pos is not None else None, scale=cfg.embed_scale)
         for key, freq in self.freqs.items():
@@ -1388,16 +1489,26 @@ class HybridEngine:
                              s.tiles[0], s.tiles[1], s.tiles[2], self.lin_tile_rows, s.B)
         return self._proj(out, w["o"], self.y[:T])
 
-    def _glu_mlp(self, f: GluMLPConfig, w: Dict[str, Any], h: torch.Tensor):
-        """-> (down(g * sigmoid(slope g) * (u + 1)), the residual gate's pre-activation W_r h)."""
+    def _glu_dense(self, f: GluMLPConfig, w: Dict[str, Any], h: torch.Tensor) -> torch.Tensor:
+        """The gated product of the gate / up projection (its epilogue), then the down projection."""
         T = h.shape[0]
         act = self.ff_act[:T * f.ff].view(T, f.ff)
-        if isinstance(w["gu"], ops.PackedWeight):
+        packed = isinstance(w["gu"], ops.PackedWeight)
+        if f.act == "gelu_tanh":
+            if packed:
+                ops.gemm(h, w["gu"], mode=2, out=act, tile_rows=w["gu"].tile_rows, n_out=f.ff, act="gelu_tanh")
+            else:
+                ops.linear(h, w["gu"], act, epilogue=5)
+        elif packed:
             ops.gemm_glu(h, w["gu"], act, f.limit, f.slope)
         else:
             ops.linear(h, w["gu"], act, epilogue=1, glu=(f.limit, f.slope))
-        r = self._proj(h, w["rg2"], self.rg[:T])
-        return self._proj(act, w["down"], self.y[:T]), r
+        return self._proj(act, w["down"], self.y[:T])
+
+    def _glu_mlp(self, f: GluMLPConfig, w: Dict[str, Any], h: torch.Tensor):
+        """-> (the feed-forward's output, the residual gate's pre-activation W_r h)."""
+        r = self._proj(h, w["rg2"], self.rg[:h.shape[0]])
+        return self._glu_dense(f, w, h), r
 
     # ---- blocks that norm sublayer outputs only ------------------------------------------------------------------
     def _forward_post(self, s: StepInputs) -> torch.Tensor:
@@ -1491,3 +1602,48 @@ class HybridEngine:
             ops.selective_scan(*scan, out_scale=m.right_scale, tiles=(s.tiles[0], s.tiles[1], s.tiles[2], self.lin_tile_rows),
                                scratch=self.scan_scratch)
         return self._proj(mix, w["o"], self.y[:T])
+
+    # ---- blocks with hyper-connections ---------------------------------------------------------------------------
+    def _forward_hyper(self, s: StepInputs) -> torch.Tensor:
+        """S copies of the stream, all equal to the embedding at the start; a sublayer reads u = sum_s in[s] x_s through its norm
+        and input convolution, and its output y enters every copy: x_t <- sum_s mix[s, t] x_s + out[t] y.  What lies between two
+        sublayers -- the update with the last one's coefficients, the read with the next one's, its norm, and in steps of single
+        rows its convolution -- is one kernel (``ops.hyper_mix_norm``); the sum of the copies goes through the final norm."""
+        cfg, w, T = self.cfg, self.w, s.T
+        x, xs, h, eps = self.x[:T], self.xs[:T], self.h[:T], cfg.eps
+        ops.embed_rows_f32(w.embed, s.ids, x, scale=cfg.embed_scale)
+        for key, freq in self.freqs.items():
+            ops.rotary_table(s.pos, freq, self.cs[key][:T], self.cs_mult[key])
+        last: Dict[str, Any] = {"x0": x}               # what enters the copies at the next boundary
+        for ri, (i, _) in enumerate(cfg.runs()):
+            L, lw = cfg.layers[i], w.layers[i]
+            self._hyper_read(last, lw, 1, (ri, "in"), s, xs, h)
+            if self.layer_tap is not None and ri > 0:
+                self.layer_tap.append(xs.sum(1))
+            y = self._mixer(ri, L, lw, s)
+            last = {"y": y, "bias": lw.get("o_b"), "mix": lw["hc1"][2], "out_c": lw["hc1"][1]}
+            if L.mlp is not None:
+                self._hyper_read(last, lw, 2, (ri, "ff"), s, xs, h)
+                y = self._glu_dense(L.mlp, lw, h)
+                last = {"y": y, "mix": lw["hc2"][2], "out_c": lw["hc2"][1]}
+        ops.hyper_mix_norm(xs, eps, h32=x, keep=False, **last)
+        if self.layer_tap is not None and cfg.runs():
+            self.layer_tap.append(x.clone())
+        return self._head(s)
+
+    def _hyper_read(self, last: Dict[str, Any], lw: Dict[str, Any], q: int, key: Tuple[int, str], s: StepInputs, xs, h) -> None:
+        """The boundary in front of sublayer q (1 mixer, 2 feed-forward): h = what the sublayer reads."""
+        T, eps = s.T, self.cfg.eps
+        args = dict(in_c=lw[f"hc{q}"][0], w=lw[f"norm{q}"], **last)
+        if not self.cfg.input_conv:
+            ops.hyper_mix_norm(xs, eps, h=h, **args)
+            return
+        cw, state = lw[f"canon{q}"], self.cache.conv.get(key)
+        if not s.multi and cw.shape[1] <= ops.HYPER_CONV_TAPS:
+            ops.hyper_mix_norm(xs, eps, h=h, conv=(cw, state, s.pos, s.slots), **args)
+            return
+        h32 = self.h32[:T]
+        ops.hyper_mix_norm(xs, eps, h32=h32, **args)
+        # (a convolution of one tap keeps no inputs: any fp32 tensor stands in for its slot)
+        ops.short_conv(h32, cw, None, state if state is not None else self.h32, s.qo_indptr, s.row_req, s.pos, s.slots, s.B, out=h,
+                       residual=True)

@@ -446,9 +446,10 @@ GEMM_ACTS = {None: 0, "relu2": 1, "gelu": 2, "gelu_tanh": 3}
 def gemm(x, w, mode: int = 0, split_k: int = 1, out=None, tile_rows: int = 128, n_out: Optional[int] = None,
          bias: Optional[torch.Tensor] = None, act: Optional[str] = None):
     """x [T, K] bf16, w [N, K] bf16 (nn.Linear.weight layout, or a PackedWeight).  bias (bf16 [N], mode 0 only) is added
-    in fp32 before the single bf16 rounding; act (mode 0 only: "relu2", "gelu", "gelu_tanh") applies to that fp32 value.
+    in fp32 before the single bf16 rounding; act ("relu2", "gelu", "gelu_tanh") applies in mode 0 to that fp32 value.
     mode 0 -> bf16 [T, N]; mode 1 -> fp32 partials [split_k, T, N]; mode 2 -> bf16 [T, n_out] = silu(gate)*up
-    with w rows packed per tile_rows-row tile (see interleave_gate_up; n_out defaults to N/2)."""
+    (with act: act(gate)*up in fp32, rounded once) with w rows packed per tile_rows-row tile (see interleave_gate_up; n_out
+    defaults to N/2)."""
     pw = _packed(w, tile_rows)
     if isinstance(x, TiledAct):
         T, K = x.T, x.K
@@ -474,7 +475,7 @@ def gemm(x, w, mode: int = 0, split_k: int = 1, out=None, tile_rows: int = 128, 
     if bias is not None:
         _need_cuda(bias)
         assert mode == 0 and bias.dtype == BF16 and bias.numel() == N and bias.is_contiguous()
-    assert act is None or mode == 0
+    assert act is None or mode in (0, 2)
     call("vb_gemm_bf16", out.data_ptr(), pw.data.data_ptr(), x_map_ptr, x_tiles_ptr, T, N, K, n_out, mode, split_k,
          tile_rows, n_out, 0, _p(bias), GEMM_ACTS[act], _stream())
     return out
@@ -1045,13 +1046,15 @@ def linear(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, epilogue: int = 
     """out [R, N] = alpha * x @ w^T with fp32 accumulation.  x [T, K] and w ([N, K], or [E, N, K] with row_off
     [E + 1] for experts) share a dtype (bf16 or fp32); out bf16 or fp32.  epilogue 1: w holds N gate rows then N up rows
     (per expert) and out = silu(gate) * up -- with glu = (limit, slope) the clamped form g = min(gate, limit),
-    u = clamp(up, -limit, limit), out = g * sigmoid(slope * g) * (u + 1); 2 / 3 / 4: out = relu(y)^2 / gelu(y) (erf) / gelu(y) (tanh form).  gather: int32 source row of x for every output row.  rows: how many rows a
-    group can have at most (grouped) / how many rows to compute (dense); default x.shape[0]."""
+    u = clamp(up, -limit, limit), out = g * sigmoid(slope * g) * (u + 1); 2 / 3 / 4: out = relu(y)^2 / gelu(y) (erf) /
+    gelu(y) (tanh form); 5: gate and up rows as for 1, out = gelu(gate) (tanh form) * up.  gather: int32 source row of x for
+    every output row.  rows: how many rows a group can have at most (grouped) / how many rows to compute (dense); default
+    x.shape[0]."""
     _need_cuda(x, w, out)
     assert x.dtype == w.dtype and x.stride(-1) == 1 and w.is_contiguous() and out.stride(-1) == 1
     groups = w.shape[0] if w.dim() == 3 else 1
     n_rows_w, K = w.shape[-2], w.shape[-1]
-    N = n_rows_w // 2 if epilogue == 1 else n_rows_w
+    N = n_rows_w // 2 if epilogue in (1, 5) else n_rows_w
     assert x.shape[1] == K and out.shape[1] >= N
     T = x.shape[0] if rows is None else rows
     call("vb_linear", out.data_ptr(), x.data_ptr(), w.data_ptr(), T, N, K, x.stride(0), out.stride(0), _dt(x), _dt(out),
@@ -1084,15 +1087,19 @@ def linear_batched(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, gate: Op
 def latent_norm_append(proj: torch.Tensor, q_off: int, c_off: int, q_rank: int, kv_rank: int, wq: torch.Tensor,
                        wc: Optional[torch.Tensor], cq_out: torch.Tensor, c_cache: Optional[torch.Tensor],
                        row_req: torch.Tensor, pos: torch.Tensor, page_indptr: torch.Tensor, page_indices: torch.Tensor,
-                       T: int, eps: float) -> None:
+                       T: int, eps: float, rot: int = 0, cs: Optional[torch.Tensor] = None, half: int = 0,
+                       layout: str = "half") -> None:
     """proj fp32 [T, ld]: the query latent at q_off is RMS-normed (wq) into cq_out [T, q_rank]; the key/value latent at
-    c_off is RMS-normed (wc) and appended to c_cache [pages, page, 1, kv_rank] (None: the layer reads another layer's)."""
+    c_off is RMS-normed (wc) and appended to c_cache [pages, page, 1, kv_rank + rot] (None: the layer reads another layer's),
+    followed by the shared key part of rot dims (the columns behind the latent), rotated on its first 2 * half dims."""
     _need_cuda(proj, cq_out)
     assert proj.dtype == F32 and proj.stride(1) == 1 and wq.dtype == F32 and cq_out.is_contiguous()
-    assert c_cache is None or (c_cache.dtype == cq_out.dtype and c_cache.is_contiguous() and wc.dtype == F32)
+    assert c_cache is None or (c_cache.dtype == cq_out.dtype and c_cache.is_contiguous() and wc.dtype == F32 and
+                               c_cache.shape[-1] == kv_rank + rot)
     call("vb_latent_norm_append", proj.data_ptr(), proj.stride(0), q_off, c_off, q_rank, kv_rank, wq.data_ptr(), _p(wc),
          cq_out.data_ptr(), _p(c_cache), row_req.data_ptr(), pos.data_ptr(), page_indptr.data_ptr(), page_indices.data_ptr(),
-         c_cache.shape[1] if c_cache is not None else 1, T, float(eps), _dt(cq_out), _stream())
+         c_cache.shape[1] if c_cache is not None else 1, T, float(eps), rot, _p(cs), half, ROTARY_LAYOUTS[layout], _dt(cq_out),
+         _stream())
 
 
 def cast_f32_bf16(src: torch.Tensor, out: torch.Tensor) -> torch.Tensor:
@@ -1124,20 +1131,26 @@ ROTARY_LAYOUTS = {"interleaved": 0, "half": 1}
 def qkv_norm_rotary_append(proj: torch.Tensor, q_off: int, k_off: int, v_off: int, cs: Optional[torch.Tensor], half: int,
                            layout: str, q_norm: Optional[torch.Tensor], k_norm: Optional[torch.Tensor], eps: float,
                            q_out: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor, row_req: torch.Tensor,
-                           pos: torch.Tensor, page_indptr: torch.Tensor, page_indices: torch.Tensor, T: int, Hq: int) -> None:
+                           pos: torch.Tensor, page_indptr: torch.Tensor, page_indices: torch.Tensor, T: int, Hq: int,
+                           bias: Optional[torch.Tensor] = None, q_scale: Optional[torch.Tensor] = None,
+                           v_norm: bool = False) -> None:
     """proj fp32 [T, ld]: Hq query heads and the key heads of k_cache [pages, page, Gk, dim] are RMS-normed over dim (weights
     fp32 [dim] shared by all heads, None: no norm), rotated on their first 2 * half dims in the given layout and written to
-    q_out / appended; the values are appended to v_cache [pages, page, Gv, vdim] as they are."""
+    q_out / appended; the values are appended to v_cache [pages, page, Gv, vdim] as they are, or (v_norm) divided by the root
+    mean square of their head.  bias (fp32, one value per q | k | v column, which then lie side by side from column 0): added
+    first.  q_scale (fp32 [Hq]): a factor per query head, applied last."""
     _need_cuda(proj, q_out, k_cache, v_cache)
     assert proj.dtype == F32 and proj.stride(1) == 1 and k_cache.dtype == q_out.dtype == v_cache.dtype
     assert k_cache.is_contiguous() and v_cache.is_contiguous() and k_cache.shape[1] == v_cache.shape[1]
     Gk, dim, Gv, vdim = k_cache.shape[2], k_cache.shape[3], v_cache.shape[2], v_cache.shape[3]
     for w in (q_norm, k_norm):
         assert w is None or (w.dtype == F32 and w.numel() == dim)
+    assert bias is None or (bias.dtype == F32 and bias.numel() >= Hq * dim + Gk * dim + Gv * vdim and q_off == 0)
+    assert q_scale is None or (q_scale.dtype == F32 and q_scale.numel() == Hq)
     call("vb_qkv_norm_rotary_append", proj.data_ptr(), proj.stride(0), q_off, k_off, v_off, _p(cs), half,
          ROTARY_LAYOUTS[layout], _p(q_norm), _p(k_norm), float(eps), q_out.data_ptr(), k_cache.data_ptr(), v_cache.data_ptr(),
          row_req.data_ptr(), pos.data_ptr(), page_indptr.data_ptr(), page_indices.data_ptr(), k_cache.shape[1], T, Hq, Gk, Gv,
-         dim, vdim, _dt(q_out), _stream())
+         dim, vdim, _dt(q_out), _p(bias), _p(q_scale), int(v_norm), _stream())
 
 
 def latent_rope_append(proj: torch.Tensor, q_off: int, c_off: int, H: int, dim: int, rot: int, kv_rank: int, wc: torch.Tensor,
@@ -1223,7 +1236,8 @@ def window_attn(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor, o
                 page_indices: torch.Tensor, T: int, H: int, G: int, dim: int, vdim: int, window: int, scale: float,
                 tiles: Optional[Tuple[torch.Tensor, torch.Tensor, torch.Tensor, int]] = None,
                 scratch: Optional[torch.Tensor] = None, rows: Optional[Tuple[torch.Tensor, int]] = None,
-                head_rows: bool = False, chunk: int = 0, k_ld: int = 0, v_ld: int = 0, v_share: int = 1) -> torch.Tensor:
+                head_rows: bool = False, chunk: int = 0, k_ld: int = 0, v_ld: int = 0, v_share: int = 1,
+                sink: Optional[torch.Tensor] = None) -> torch.Tensor:
     """gate: an fp32 view [T, H * vdim] (any row stride) or None.  tiles = (qo_indptr, tile_req, tile_row0, n_tiles):
     run the tiled prompt kernel over those row tiles instead of the per-row kernel.  scratch (fp32): lets the per-row kernel
     split a row's keys over several CTAs when the step has few rows.  rows = (int32 row indices, count): serve only those
@@ -1231,8 +1245,10 @@ def window_attn(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor, o
     heads that share a key/value head (many heads on few key/value heads: latent attention).  chunk > 0: a position sees
     only the keys of its own block of `chunk` positions.  k_ld / v_ld: elements per token of the key / value cache when they
     are not G * dim / G * vdim (values that are a leading slice of the key rows).  v_share: consecutive key heads reading one
-    value head.  An fp32 ``out`` beside bf16 operands is written in fp32."""
+    value head.  An fp32 ``out`` beside bf16 operands is written in fp32.  sink (fp32 [H]): exp(sink[h]) joins the denominator of
+    head h's softmax."""
     _need_cuda(q, k_cache, v_cache, out)
+    assert sink is None or (sink.dtype == F32 and sink.numel() == H)
     out_f32 = int(out.dtype == F32)
     ld_gate = gate.stride(0) if gate is not None else 0
     if tiles is None:
@@ -1241,13 +1257,13 @@ def window_attn(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor, o
              row_req.data_ptr(), pos.data_ptr(), page_indptr.data_ptr(), page_indices.data_ptr(), n, H, G, dim, vdim,
              k_cache.shape[1], int(window), float(scale), _dt(q), _p(scratch), scratch.numel() if scratch is not None else 0,
              _p(rows[0]) if rows is not None else None, int(head_rows), int(chunk), int(k_ld), int(v_ld), int(v_share), out_f32,
-             _stream())
+             _p(sink), _stream())
     else:
         qo, tile_req, tile_row0, n_tiles = tiles
         call("vb_window_attn_tiled", out.data_ptr(), q.data_ptr(), k_cache.data_ptr(), v_cache.data_ptr(), _p(gate),
              ld_gate, pos.data_ptr(), page_indptr.data_ptr(), page_indices.data_ptr(), qo.data_ptr(), tile_req.data_ptr(),
              tile_row0.data_ptr(), n_tiles, T, H, G, dim, vdim, k_cache.shape[1], int(window), float(scale), _dt(q),
-             int(chunk), int(k_ld), int(v_ld), int(v_share), out_f32, _stream())
+             int(chunk), int(k_ld), int(v_ld), int(v_share), out_f32, _p(sink), _stream())
     return out
 
 
@@ -1434,6 +1450,35 @@ def short_conv(x: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor], s
          out_f32.stride(0) if out_f32 is not None else 0, x.data_ptr(), x.stride(0), w.data_ptr(), _p(bias), state.data_ptr(),
          qo_indptr.data_ptr(), row_req.data_ptr(), pos.data_ptr(), slots.data_ptr(), T, B, C, taps, 1 if act == "silu" else 0,
          int(residual), _dt(out) if out is not None else 1, _stream())
+
+
+HYPER_CONV_TAPS = 4        # the longest convolution that hyper_mix_norm runs by itself
+
+
+def hyper_mix_norm(xs: torch.Tensor, eps: float, x0: Optional[torch.Tensor] = None, y: Optional[torch.Tensor] = None,
+                   bias: Optional[torch.Tensor] = None, mix: Optional[torch.Tensor] = None, out_c: Optional[torch.Tensor] = None,
+                   in_c: Optional[torch.Tensor] = None, w: Optional[torch.Tensor] = None, h: Optional[torch.Tensor] = None,
+                   h32: Optional[torch.Tensor] = None, conv: Optional[Tuple] = None, keep: bool = True) -> None:
+    """One boundary between sublayers of a stack with hyper-connections, in place on the copies xs [T, S, W] (fp32):
+    x_t <- sum_s mix[s, t] x_s + out_c[t] (y + bias) -- or, with x0 [T, W], every copy starts as that row --, then
+    u = sum_s in_c[s] x_s (None: ones) and, with a norm weight w, h = u / rms(u) * w to h (bf16 or fp32) and / or h32; without
+    one, h32 = u.  conv = (weights [W, taps], state [slots, taps - 1, W], pos, slots): row t is request t's only row, and
+    h <- h + conv(h) with that slot's last inputs.  keep False: the new copies are not written back."""
+    _need_cuda(xs)
+    T, S, W = xs.shape
+    assert xs.dtype == F32 and xs.is_contiguous()
+    for t in (x0, y, h32):
+        assert t is None or (t.dtype == F32 and t.is_contiguous() and tuple(t.shape) == (T, W))
+    for t, n in ((bias, W), (mix, S * S), (out_c, S), (in_c, S), (w, W)):
+        assert t is None or (t.dtype == F32 and t.is_contiguous() and t.numel() == n)
+    assert h is None or (h.is_contiguous() and tuple(h.shape) == (T, W))
+    cw, cst, pos, slots = conv if conv is not None else (None, None, None, None)
+    if cw is not None:
+        assert cw.dtype == F32 and cw.is_contiguous() and cw.shape[0] == W and pos.numel() >= T and slots.numel() >= T
+        assert cw.shape[1] == 1 or (cst.dtype == F32 and cst.is_contiguous() and tuple(cst.shape[1:]) == (cw.shape[1] - 1, W))
+    call("vb_hyper_mix_norm", xs.data_ptr(), S, _p(x0), _p(y), _p(bias), _p(mix), _p(out_c), _p(in_c), _p(w), _p(h), _p(h32), T, W,
+         float(eps), _p(cw), cw.shape[1] if cw is not None else 1, _p(cst), _p(pos), _p(slots), int(keep),
+         _dt(h) if h is not None else 1, _stream())
 
 
 def cast_rows(src: torch.Tensor, out: torch.Tensor) -> torch.Tensor:
