@@ -17,6 +17,12 @@ rotated key part, own and shared cached rows; pooled-window sigmoid attention be
 router over clamped gated experts; tied head) beside Bobavik (window attention, linear attention with a recurrent state,
 mixture of experts) at equal width, head count, head size and expert width per token.
 
+``--arch zopipel``: the Zopipel design (four hyper-connected copies of the stream, input convolutions on both sublayers; windowed
+latent attention with a query latent and a shared rotated key part; grouped-head attention with biases, unit-RMS values and a
+softmax sink; gated gelu feed-forward) beside its closest relative on the same engine, Fovunex (latent attention with a shared
+rotated key part, gated residuals, gated dense feed-forward) with as many latent-attention and softmax-attention layers, at equal
+width, head count, head size and feed-forward width -- and beside Bobavik with attention layers only.
+
 Per size and engine: prefill of one 1024-token prompt (eager launches) and one decode step of 32 requests at context 512
 (a CUDA-graph replay, as served), timed with CUDA events after warm-up; an L2-sized buffer is overwritten between timed
 iterations.  Output: one JSON line per size.
@@ -88,6 +94,32 @@ def nadevik_config(width: int, ff: int, experts: int = 8, top: int = 3) -> dict:
             "embedding": {"scale": 1.0, "bigram": {"buckets": 8191, "mul_prev": 31, "mul_cur": 7}}, "layers": layers}
 
 
+def zopipel_config(width: int, ff: int) -> dict:
+    """four layers: latent attention, attention, attention, latent attention, each with a feed-forward; 128-wide heads (latent
+    attention: 128 unrotated + 64 rotated dims on a latent of 128, query latent of 3/8 of the width, window 4096; attention: a
+    quarter as many key/value heads, 128-wide keys and values, rotated whole), four copies of the stream, convolutions of 4
+    taps, a dense feed-forward as wide as the experts a Bobavik token uses; no looped span (every layer once)"""
+    heads = width // 128
+    lat = {"heads": heads, "dim": 128, "rot_dim": 64, "vdim": 128, "kv_rank": 128, "q_rank": width * 3 // 8, "scale": 192 ** -0.5,
+           "mask": {"size": 4096}, "rot": {"base": 1e4, "dims": 64}}
+    att = {"heads": heads, "kv_heads": max(1, heads // 4), "dim": 128, "vdim": 128, "scale": 128 ** -0.5,
+           "rot": {"dims": 128, "base": 1e6, "scaling": {"factor": 4.0}}}
+    mlp = {"kind": "dense", "ff": 3 * ff}
+    layers = [{"type": t, "mixer": dict(lat if t == "latent_attention" else att), "mlp": dict(mlp)}
+              for t in ("latent_attention", "attention", "attention", "latent_attention")]
+    return {"architecture": "Zopipel", "width": width, "vocab": VOCAB, "norm": {"eps": 1e-6}, "streams": 4, "canon": {"taps": 4},
+            "layers": layers}
+
+
+def fovunex_attention_config(width: int, ff: int) -> dict:
+    """Fovunex as Zopipel's neighbour: latent attention, two-map attention, two-map attention, latent attention, each with a
+    feed-forward (the two maps of 64 dims make 128 query / key dims per head)"""
+    c = fovunex_config(width, ff)
+    lat, att = c["layers"][0], c["layers"][2]
+    c["layers"] = [lat, att, att, lat]
+    return c
+
+
 def bobavik_config(width: int, ff: int, experts: int = 8, top: int = 2, window: int = 4096,
                    kinds=("attention", "lightning", "lightning", "attention")) -> dict:
     heads = width // 128
@@ -137,8 +169,13 @@ def bench_bobavik(width: int, ff: int, steps: int, warmup: int, flush, kinds=Non
     from vox_serve_b200.model.fovunex import FovunexModel
     from vox_serve_b200.model.nadevik import NadevikModel
     from vox_serve_b200.model.razevik import RazevikModel
+    from vox_serve_b200.model.zopipel import ZopipelModel
 
-    if design == "nadevik":
+    if design == "zopipel":
+        model = ZopipelModel("zopipel-synthetic:1", config=zopipel_config(width, ff), device="cuda:0")
+    elif design == "fovunex_attention":
+        model = FovunexModel("fovunex-synthetic:1", config=fovunex_attention_config(width, ff), device="cuda:0")
+    elif design == "nadevik":
         model = NadevikModel("nadevik-synthetic:1", config=nadevik_config(width, ff), device="cuda:0")
     elif design == "fovunex":
         model = FovunexModel("fovunex-synthetic:1", config=fovunex_config(width, ff), device="cuda:0")
@@ -241,6 +278,19 @@ def run(sizes, steps: int, warmup: int, only: str = "", arch: str = "bobavik") -
                 line["fovunex"] = bench_bobavik(width, ff, steps, warmup, flush, design="fovunex")
             if only in ("", "bobavik"):
                 line["bobavik"] = bench_bobavik(width, ff, steps, warmup, flush)
+            print(json.dumps(line), flush=True)
+            torch.cuda.empty_cache()
+            continue
+        if arch == "zopipel":
+            line = {"bench": "zopipel_vs_fovunex", "width": width, "layers": LAYERS, "prompt": PROMPT, "decode_batch": BATCH,
+                    "context": CONTEXT, "steps": steps, "warmup": warmup, "dtype": "bf16", "data": "synthetic",
+                    "l2": "192 MiB buffer overwritten between timed iterations"}
+            if only in ("", "zopipel"):
+                line["zopipel"] = bench_bobavik(width, ff, steps, warmup, flush, design="zopipel")
+            if only in ("", "fovunex"):
+                line["fovunex"] = bench_bobavik(width, ff, steps, warmup, flush, design="fovunex_attention")
+            if only in ("", "bobavik"):
+                line["bobavik_attention"] = bench_bobavik(width, ff, steps, warmup, flush, kinds=("attention",) * LAYERS)
             print(json.dumps(line), flush=True)
             torch.cuda.empty_cache()
             continue

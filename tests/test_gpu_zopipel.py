@@ -1,0 +1,761 @@
+"""Zopipel on the hybrid engine against the plain float64 oracle (tests/zopipel_oracle.py): every mechanism alone, whole prompts
+against token-by-token decoding, portions of several sizes, batches against single requests, reuse of pages and slots, keys
+far away / at page borders / just inside and outside a window with inputs built so that a wrong key (or a missing sink) shows,
+convolution state on reused slots, other sizes, and greedy generation through ModelWorker + Scheduler.  Small configurations
+with random weights; float32 is compared tightly, bfloat16 loosely.
+"""
+import json
+import os
+import tempfile
+
+import pytest
+import torch
+
+from tests import zopipel_oracle as O
+
+F32, BF16, I32, F64 = torch.float32, torch.bfloat16, torch.int32, torch.float64
+DEV = "cuda"
+
+
+# ---- CPU: configuration, registry, cache, the oracle's own rules ------------------------------------------------------
+def test_config_reader_covers_every_branch():
+    from vox_serve_b200._lib import VoxB200Error
+    from vox_serve_b200.hybrid_engine import GluMLPConfig, LatentAttentionConfig, WindowAttentionConfig
+    from vox_serve_b200.model.zopipel import zopipel_config
+
+    c = zopipel_config(O.make_config())
+    assert (c.block, c.norm, c.eps, c.streams, c.input_conv, c.tied_head, c.embed_scale) == ("hyper", "rmsnorm", 1e-5, 2, 3, False, 1.0)
+    assert [L.kind for L in c.layers] == ["latent", "attention", "latent", "attention", "attention"]
+    lat, att = c.layers[0].mixer, c.layers[1].mixer
+    assert isinstance(lat, LatentAttentionConfig) and isinstance(att, WindowAttentionConfig)
+    assert (lat.heads, lat.dim, lat.rot_dim, lat.vdim, lat.kv_rank, lat.q_rank, lat.scale, lat.window) == (3, 8, 6, 10, 12, 20, 0.27, 11)
+    assert lat.head_gate and not lat.value_gate and lat.kv_from is None
+    assert (lat.rotary.dims, lat.rotary.base, lat.rotary.layout, lat.rotary.factor) == (6, 300.0, "half", None)
+    assert (att.heads, att.kv_heads, att.dim, att.vdim, att.scale, att.window, att.sink) == (4, 2, 12, 6, 0.33, 0, 0.0)
+    assert att.bias and att.value_norm and att.head_factor and not att.gate and not att.v_mix
+    assert (att.rotary.dims, att.rotary.base, att.rotary.layout, att.rotary.factor, att.rotary.scaling) == (8, 500.0, "half", 4.0, "linear")
+    assert isinstance(c.layers[0].mlp, GluMLPConfig) and (c.layers[0].mlp.ff, c.layers[0].mlp.act) == (40, "gelu_tanh")
+    assert c.layers[2].mlp is None
+    assert c.runs() == [(0, False), (1, False), (2, False), (1, True), (2, False), (1, True), (2, False), (3, False), (4, False)]
+    # what a configuration may leave out
+    c2 = zopipel_config(O.make_config(canon=0, loop=None, l_rot=0, l_window=0, a_rot_dims=0, a_window=7, streams=1))
+    assert c2.input_conv == 0 and c2.runs() == [(i, False) for i in range(5)] and c2.layers[0].mixer.rotary is None
+    assert c2.layers[0].mixer.window == 0 and c2.layers[1].mixer.window == 7 and c2.layers[1].mixer.rotary is None
+    c3 = zopipel_config(O.make_config(a_factor=None))
+    assert c3.layers[1].mixer.rotary.factor is None
+    bad = O.make_config()
+    bad["layers"][0]["type"] = "convolution"
+    with pytest.raises(VoxB200Error):
+        zopipel_config(bad)
+    with pytest.raises(VoxB200Error):
+        zopipel_config(O.make_config(a_heads=3, a_kv_heads=2))
+    with pytest.raises(VoxB200Error):
+        zopipel_config(O.make_config(l_rot=4, l_rot_dims=6))
+    with pytest.raises(VoxB200Error):
+        zopipel_config(O.make_config(a_rot_dims=14))
+    with pytest.raises(VoxB200Error):
+        zopipel_config(O.make_config(loop=(1, 9, 2)))
+
+
+def test_rotary_frequencies_linear_scaling():
+    from vox_serve_b200.hybrid_engine import RotaryConfig
+
+    r = {"dims": 10, "base": 700.0, "scaling": {"factor": 2.5}}
+    assert RotaryConfig(10, 700.0, 2.5, layout="half", scaling="linear").frequencies().tolist() == pytest.approx(O.rotation_angles(r), rel=1e-14)
+    assert RotaryConfig(10, 700.0, layout="half", scaling="linear").frequencies().tolist() == pytest.approx(
+        O.rotation_angles({"dims": 10, "base": 700.0}), rel=1e-14)
+
+
+def test_registry_and_cache():
+    from vox_serve_b200.build import PROFILES
+    from vox_serve_b200.hybrid_engine import HybridCache
+    from vox_serve_b200.model import build_profile, get_model_class
+    from vox_serve_b200.model.zopipel import ZopipelModel, zopipel_config
+
+    cfg = O.make_config()
+    with tempfile.TemporaryDirectory() as d:
+        with open(os.path.join(d, "config.json"), "w") as f:
+            json.dump(cfg, f)
+        assert get_model_class(d) is ZopipelModel and build_profile(d) == "text_hyper" and "hyper.cu" in PROFILES["text_hyper"]
+    assert get_model_class("zopipel-synthetic:3") is ZopipelModel
+    cache = HybridCache(zopipel_config(cfg), 5, 8, 3, torch.float32, "cpu")
+    assert sorted(cache.k) == list(range(9)) and not cache.state              # one cache per run of a looped layer
+    assert tuple(cache.k[0].shape) == (5, 8, 1, 18) and cache.k[0].data_ptr() == cache.v[0].data_ptr()
+    assert tuple(cache.k[1].shape) == (5, 8, 2, 12) and tuple(cache.v[1].shape) == (5, 8, 2, 6)
+    assert len({cache.k[i].data_ptr() for i in range(9)}) == 9
+    # the convolutions' inputs: mixer and feed-forward of every run; layers without a feed-forward have one
+    assert sorted(cache.conv) == sorted([(i, "in") for i in range(9)] + [(i, "ff") for i in (0, 1, 3, 5, 7)])
+    assert tuple(cache.conv[(0, "ff")].shape) == (3, 2, 48) and cache.conv[(1, "in")].data_ptr() != cache.conv[(3, "in")].data_ptr()
+    assert not HybridCache(zopipel_config(O.make_config(canon=1)), 5, 8, 3, torch.float32, "cpu").conv
+
+
+def test_oracle_mechanisms_by_hand():
+    assert O.visible(4, 2).tolist() == [[True, False, False, False], [True, True, False, False], [False, True, True, False],
+                                        [False, False, True, True]]
+    assert O.visible(3, 0).tolist() == [[True, False, False], [True, True, False], [True, True, True]]
+    s = torch.tensor([[0.0, 0.0], [0.0, 0.0]], dtype=F64)
+    assert torch.allclose(O.softmax_rows(s, O.visible(2, 0), True), torch.tensor([[0.5, 0.0], [1 / 3, 1 / 3]], dtype=F64))
+    assert torch.allclose(O.softmax_rows(s, O.visible(2, 0), False), torch.tensor([[1.0, 0.0], [0.5, 0.5]], dtype=F64))
+    assert O.layer_order({"layers": [0] * 4, "loop": {"start": 1, "stop": 3, "times": 2}}) == [0, 1, 2, 1, 2, 3]
+    x = [torch.tensor([[1.0]], dtype=F64), torch.tensor([[10.0]], dtype=F64)]
+    mix, out = torch.tensor([[1.0, 2.0], [3.0, 4.0]], dtype=F64), torch.tensor([5.0, 6.0], dtype=F64)
+    assert [float(t) for t in O.write_streams(x, torch.tensor([[100.0]], dtype=F64), mix, out)] == [531.0, 642.0]     # [from, to]
+    assert float(O.read_streams(x, torch.tensor([2.0, 3.0], dtype=F64))) == 32.0
+    u = torch.tensor([[1.0], [2.0], [4.0]], dtype=F64)
+    assert O.causal_conv(u, torch.tensor([[10.0, 1.0]], dtype=F64)).view(-1).tolist() == [1.0, 12.0, 24.0]
+
+
+# ---- helpers ---------------------------------------------------------------------------------------------------------
+def _worker(cfg, sd, dtype, slots=3, pages=24, page_size=8, max_rows=256, **kw):
+    from vox_serve_b200.model.zopipel import ZopipelModel
+    from vox_serve_b200.worker import ModelWorker
+
+    model = ZopipelModel("zopipel-test", dtype=dtype, device="cuda:0", state_dict=sd, config=cfg, max_tokens=512, **kw)
+    return ModelWorker("zopipel-test", max_batch_size=slots, max_num_pages=pages, page_size=page_size, model=model,
+                       max_prefill_tokens=max_rows, max_logit_rows=max_rows)
+
+
+def _replay(worker, seqs, steps, free=True):
+    """steps: [[(id, count), ...], ...]; every token's logits are tapped.  Returns id -> [len, vocab] fp32 (CPU)."""
+    from vox_serve_b200.requests import Request
+
+    live, at, out = {}, {k: 0 for k in seqs}, {k: [] for k in seqs}
+    for step in steps:
+        reqs = []
+        for rid, n in step:
+            toks = seqs[rid][at[rid]:at[rid] + n]
+            if rid not in live:
+                live[rid] = Request(request_id=rid, prompt=list(toks))
+            else:
+                live[rid].pending_tokens = (live[rid].pending_tokens or []) + list(toks)
+            live[rid].step_tokens, live[rid].logit_rows = n, list(range(n))
+            at[rid] += n
+            reqs.append(live[rid])
+        inp = worker.prepare_lm_inputs(reqs, [])
+        assert inp is not None and len(reqs) == len(step), [r.finish_reason for r in live.values()]
+        task = (worker.run_lm_prefill if inp["is_prefill"] else worker.run_lm_decode)(reqs, inp)
+        try:
+            while True:
+                task.send(None)
+        except StopIteration:
+            pass
+        for rid, _ in step:
+            out[rid].append(worker.step_logits(rid))
+        for rid, _ in step:
+            if free and at[rid] == len(seqs[rid]):
+                live[rid].done_all = True
+                worker.free_kv_cache(live.pop(rid))
+    return {k: torch.cat(v, 0) for k, v in out.items() if v}
+
+
+def _err(got, ref):
+    """difference over the vocabulary (mean removed), rms, relative to the rms of the reference logits; the worst position"""
+    d = got.double() - ref
+    d = d - d.mean(-1, keepdim=True)
+    r = ref - ref.mean(-1, keepdim=True)
+    return (d.pow(2).mean(-1).sqrt() / r.pow(2).mean().sqrt()).max().item()
+
+
+TOL = {F32: 1e-4, BF16: 8e-2}
+
+
+def _tokens(n, vocab, seed):
+    g = torch.Generator().manual_seed(seed)
+    return torch.randint(0, vocab, (n,), generator=g).tolist()
+
+
+# ---- whole models ----------------------------------------------------------------------------------------------------
+@pytest.mark.gpu
+@pytest.mark.parametrize("dtype", [F32, BF16])
+def test_layers_and_logits_whole_prompt(dtype):
+    cfg = O.make_config()
+    sd = O.make_weights(cfg, 3)
+    toks = _tokens(45, cfg["vocab"], 5)
+    w = _worker(cfg, sd, dtype)
+    w.engine.layer_tap = []
+    got = _replay(w, {"a": toks}, [[("a", 45)]])["a"]
+    taps, w.engine.layer_tap = w.engine.layer_tap, None
+    layers = []
+    ref = O.forward(cfg, sd, toks, layers)
+    assert len(taps) == len(layers) == 9
+    for i, (x, r) in enumerate(zip(taps, layers)):
+        rel = (x.cpu().double() - r).pow(2).mean(-1).sqrt() / r.pow(2).mean().sqrt()        # per token
+        assert rel.max().item() < (1e-5 if dtype == F32 else 6e-2), (i, rel.max().item())
+    assert _err(got, ref) < TOL[dtype]
+
+
+@pytest.mark.gpu
+@pytest.mark.parametrize("layers,loop", [(("latent",), None), (("latent-",), None), (("attn",), None), (("attn-",), None),
+                                         (("attn-", "latent-"), (0, 2, 2)), (("latent",), (0, 1, 4)), (("attn",), (0, 1, 1)),
+                                         (("attn", "latent", "latent-"), (2, 3, 3))])
+def test_each_mixer_alone(layers, loop):
+    cfg = O.make_config(layers=layers, loop=loop)
+    sd = O.make_weights(cfg, 11)
+    toks = _tokens(30, cfg["vocab"], 2)
+    got = _replay(_worker(cfg, sd, F32), {"a": toks}, [[("a", 30)]])["a"]
+    assert _err(got, O.forward(cfg, sd, toks)) < TOL[F32]
+
+
+OTHER_SIZES = [
+    dict(l_heads=1, a_heads=1, a_kv_heads=1, streams=1, loop=None),
+    dict(l_heads=5, a_heads=6, a_kv_heads=6, a_dim=5, a_vdim=9, a_rot_dims=4, streams=3, canon=2),
+    dict(a_heads=6, a_kv_heads=1, a_dim=16, a_vdim=16, a_rot_dims=16, l_dim=16, l_vdim=4, l_rank=7, l_q_rank=9, width=44, ff=20),
+    dict(l_rot=0, l_window=1, a_window=1, canon=1, a_rot_dims=0, ff=3),
+    dict(l_rot=8, l_rot_dims=4, l_window=0, canon=0, a_factor=None, streams=4),
+    dict(l_window=5, a_window=9, canon=6, streams=5, loop=(0, 4, 2), width=50, eps=1e-2),
+    dict(l_heads=18, a_heads=34, a_kv_heads=2, a_dim=4, a_vdim=3, a_rot_dims=2, l_dim=4, l_rot=2, l_vdim=3, l_rank=24, l_q_rank=8, canon=4),
+    dict(width=37, vocab=31, streams=2, canon=3, l_rank=11, l_rot=2, l_dim=1, l_vdim=1, a_dim=2, a_vdim=1, a_rot_dims=2),
+    dict(a_base=12.0, a_factor=1.0, l_base=9.0, l_window=40, streams=7, canon=5, a_kv_heads=4),
+]
+
+
+@pytest.mark.gpu
+@pytest.mark.parametrize("kw", OTHER_SIZES)
+def test_other_sizes(kw):
+    """head counts of one and many, key/value heads = heads and = 1, key size != value size, sizes of one and odd sizes that rule
+    tensor-core projections and 16-byte rows out, windows of one / none (on both mixers), no rotated part and rotation on a slice,
+    scaling by one and none, convolutions of no tap, one and more taps than the fused form takes, one to seven streams, loops of
+    several spans, a large eps."""
+    cfg = O.make_config(layers=("latent", "attn", "latent-", "attn-"), **{"loop": (1, 3, 2), **kw})
+    sd = O.make_weights(cfg, 7)
+    toks = _tokens(41, cfg["vocab"], 3)
+    ref = O.forward(cfg, sd, toks)
+    cuts = [[("a", 17)], [("a", 2)], [("a", 9)]] + [[("a", 1)]] * 13
+    w = _worker(cfg, sd, F32)
+    assert _err(_replay(w, {"a": toks}, [[("a", 41)]])["a"], ref) < TOL[F32]
+    assert _err(_replay(w, {"a": toks}, cuts)["a"], ref) < TOL[F32]
+    assert _err(_replay(_worker(cfg, sd, BF16), {"a": toks}, cuts)["a"], ref) < TOL[BF16]
+
+
+@pytest.mark.gpu
+@pytest.mark.parametrize("dtype", [F32, BF16])
+def test_prefill_decode_portions_and_batches(dtype):
+    """whole prompt = token by token from the first token = portions of 1 ... 64 tokens cut inside pages and windows = batches of
+    five unequal requests on three slots with requests left out of steps and reused pages and slots."""
+    cfg = O.make_config()
+    sd = O.make_weights(cfg, 5)
+    V = cfg["vocab"]
+    seqs = {k: _tokens(n, V, i) for i, (k, n) in enumerate((("a", 70), ("b", 9), ("c", 33), ("d", 1), ("e", 26)))}
+    ref = {k: O.forward(cfg, sd, t) for k, t in seqs.items()}
+    w = _worker(cfg, sd, dtype, pages=40)
+    same = (lambda k: 2e-5 * ref[k].abs().max().item()) if dtype == F32 else (lambda k: 0.15 * ref[k].abs().max().item())
+    whole = _replay(w, seqs, [[(k, len(t))] for k, t in seqs.items()])
+    for k in seqs:
+        assert _err(whole[k], ref[k]) < TOL[dtype], k
+    one = _replay(w, {"a": seqs["a"]}, [[("a", 1)]] * 70)["a"]
+    assert _err(one, ref["a"]) < TOL[dtype] and (one - whole["a"]).abs().max().item() < same("a")
+    for cuts in ([2] * 35, [2, 2, 3, 1, 5, 7, 11, 13, 2, 24], [64, 2, 4], [3, 64, 3], [8, 8, 8, 8, 8, 8, 8, 8, 6], [9, 4, 4, 53]):
+        assert sum(cuts) == 70
+        got = _replay(w, {"a": seqs["a"]}, [[("a", n)] for n in cuts])["a"]
+        assert _err(got, ref["a"]) < TOL[dtype] and (got - whole["a"]).abs().max().item() < same("a"), cuts
+    # five requests on three slots: portions beside single tokens, requests left out of steps, slots and pages taken again
+    steps = [[("a", 5), ("b", 2)], [("a", 1), ("b", 1), ("c", 20)], [("b", 6), ("c", 1)], [("a", 30), ("c", 12)],
+             [("a", 1)], [("d", 1), ("a", 2)], [("e", 3), ("a", 31)], [("e", 1)], [("e", 22)]]
+    got = _replay(w, seqs, steps)
+    for k in seqs:
+        assert _err(got[k], ref[k]) < TOL[dtype] and (got[k] - whole[k]).abs().max().item() < same(k), k
+    assert w.empty_pages.qsize() == 40 and len(w.free_slots) == 3
+
+
+@pytest.mark.gpu
+@pytest.mark.parametrize("canon", [4, 6])
+def test_long_decoding_across_pages_and_windows(canon):
+    """(six taps: the convolution runs as a kernel of its own in single-token steps too)"""
+    cfg = O.make_config(canon=canon, layers=("latent", "attn", "latent-"), loop=(0, 2, 2))
+    sd = O.make_weights(cfg, 9)
+    toks = _tokens(250, cfg["vocab"], 4)
+    ref = O.forward(cfg, sd, toks)
+    for graph in (True, False):
+        w = _worker(cfg, sd, F32, pages=40)
+        w.use_cuda_graph = graph
+        got = _replay(w, {"a": toks}, [[("a", 10)]] + [[("a", 1)]] * 240)["a"]
+        assert _err(got, ref) < TOL[F32], graph
+
+
+@pytest.mark.gpu
+def test_decoding_batches_on_reused_slots():
+    """steps of single tokens only, four requests on two slots one after the other, beside ones that stay: what a slot's
+    convolutions and pages held before never shows"""
+    cfg = O.make_config(canon=4, layers=("latent", "attn"), loop=None, streams=3)
+    sd = O.make_weights(cfg, 15)
+    seqs = {k: _tokens(n, cfg["vocab"], 20 + i) for i, (k, n) in enumerate((("a", 40), ("b", 3), ("c", 17), ("d", 2), ("e", 9)))}
+    w = _worker(cfg, sd, F32, slots=2, pages=9)
+    steps = [[("a", 1), ("b", 1)]] * 3 + [[("c", 1), ("a", 1)]] * 17 + [[("a", 1), ("d", 1)]] * 2 + [[("e", 1), ("a", 1)]] * 9 + [[("a", 1)]] * 9
+    got = _replay(w, seqs, steps)
+    for k in seqs:
+        assert _err(got[k], O.forward(cfg, sd, seqs[k])) < TOL[F32], k
+    assert w.empty_pages.qsize() == 9 and len(w.free_slots) == 2
+
+
+@pytest.mark.gpu
+def test_bfloat16_tensor_core_sizes():
+    """sizes whose projections run on the tensor-core kernels (multiples of 8 / 16 / 64): a 600-token prompt whole (tiled
+    attention) against portions (single rows among them), the plain projection kernel and the oracle"""
+    cfg = O.make_config(layers=("latent", "attn", "latent"), loop=(1, 2, 2), width=128, vocab=160, streams=4, canon=3, l_heads=4,
+                        l_dim=32, l_rot=16, l_vdim=32, l_rank=64, l_q_rank=48, l_window=100, a_heads=4, a_kv_heads=2, a_dim=32,
+                        a_vdim=32, a_rot_dims=32, ff=192)
+    sd = O.make_weights(cfg, 21)
+    toks = _tokens(600, cfg["vocab"], 6)
+    ref = O.forward(cfg, sd, toks)
+    kw = dict(slots=2, pages=24, page_size=64, max_rows=1024)
+    cuts = [[("a", 130)], [("a", 1)], [("a", 300)], [("a", 2)], [("a", 167)]]
+    w = _worker(cfg, sd, BF16, **kw)
+    whole, parts = _replay(w, {"a": toks}, [[("a", 600)]])["a"], _replay(w, {"a": toks}, cuts)["a"]
+    plain = _replay(_worker(cfg, sd, BF16, tensor_core_projections=False, **kw), {"a": toks}, [[("a", 600)]])["a"]
+    for got in (whole, parts, plain):
+        assert _err(got, ref) < TOL[BF16]
+    w32 = _worker(cfg, sd, F32, **kw)
+    assert _err(_replay(w32, {"a": toks}, [[("a", 600)]])["a"], ref) < TOL[F32]
+    w32.engine.use_tiled_attention = False
+    assert _err(_replay(w32, {"a": toks}, [[("a", 333)], [("a", 267)]])["a"], ref) < TOL[F32]
+
+
+# ---- single mechanisms -----------------------------------------------------------------------------------------------
+def _paged(n_req_tokens, page_size, seed=0, spare=3):
+    """scattered pages for requests of the given lengths -> (page_indptr, page_indices, number of pages)"""
+    need = [(n + page_size - 1) // page_size for n in n_req_tokens]
+    total = sum(need) + spare
+    perm = torch.randperm(total, generator=torch.Generator().manual_seed(seed)).tolist()
+    indptr, idx = [0], []
+    for n in need:
+        idx += perm[len(idx):len(idx) + n]
+        indptr.append(len(idx))
+    return torch.tensor(indptr, dtype=I32, device=DEV), torch.tensor(idx, dtype=I32, device=DEV), total
+
+
+def _step_tables(spans):
+    """spans: per request (first position, rows) -> qo_indptr, row_req, pos (device int32)"""
+    qo, row_req, pos = [0], [], []
+    for b, (p0, n) in enumerate(spans):
+        row_req += [b] * n
+        pos += list(range(p0, p0 + n))
+        qo.append(qo[-1] + n)
+    mk = lambda v: torch.tensor(v, dtype=I32, device=DEV)
+    return mk(qo), mk(row_req), mk(pos)
+
+
+def _gather(cache, indptr, pages, b, n):
+    """the first n cached rows of request b -> float64 [n, heads, dims] (CPU)"""
+    ps = cache.shape[1]
+    pg = pages[int(indptr[b]):int(indptr[b + 1])].tolist()
+    return torch.stack([cache[pg[t // ps], t % ps] for t in range(n)]).double().cpu()
+
+
+@pytest.mark.gpu
+@pytest.mark.parametrize("dtype", [F32, BF16])
+@pytest.mark.parametrize("S,W", [(1, 48), (2, 37), (3, 64), (4, 1030), (4, 2048), (5, 40), (16, 12)])
+def test_hyper_connections_start_update_read_end(dtype, S, W):
+    """the copies over four sublayers with biases and asymmetric mixing matrices: few rows and many, widths that move in 16-byte
+    pieces and that do not, 1 ... 16 copies; the read of a sublayer, the copies themselves, and the sum at the end"""
+    from vox_serve_b200 import ops
+
+    for T in (3, 200):
+        g = torch.Generator().manual_seed(S * 100 + T)
+        r = lambda *s: torch.randn(*s, generator=g, dtype=F32)
+        dev = lambda t: t.to(DEV).contiguous()
+        e = r(T, W)
+        xs = torch.full((T, S, W), float("nan"), dtype=F32, device=DEV)
+        ref = [e.double()] * S
+        last, tol = {"x0": dev(e)}, (1e-5 if dtype == F32 else 2e-2)
+        for k in range(4):
+            a, w, eps = r(S), r(W), 1e-4
+            h = torch.zeros(T, W, dtype=dtype, device=DEV)
+            h32 = torch.zeros(T, W, dtype=F32, device=DEV)
+            ops.hyper_mix_norm(xs, eps, in_c=dev(a), w=dev(w), h=h, h32=h32 if k % 2 else None, **last)
+            want = O.rms_norm(O.read_streams(ref, a.double()), w.double(), eps)
+            assert (h.double().cpu() - want).abs().max().item() < tol * max(1.0, want.abs().max().item()), k
+            if k % 2:
+                assert (h32.double().cpu() - want).abs().max().item() < 2e-5 * max(1.0, want.abs().max().item()), k
+            big = max(1.0, max(x.abs().max().item() for x in ref))
+            for s in range(S):
+                assert (xs[:, s].double().cpu() - ref[s]).abs().max().item() < 1e-5 * big, (k, s)
+            y, b, mix, out = r(T, W), (r(W) if k != 1 else None), r(S, S) * 0.4, r(S)
+            last = {"y": dev(y), "bias": dev(b) if b is not None else None, "mix": dev(mix), "out_c": dev(out)}
+            ref = O.write_streams(ref, y.double() + (b.double() if b is not None else 0.0), mix.double(), out.double())
+        before, total = xs.clone(), torch.zeros(T, W, dtype=F32, device=DEV)
+        ops.hyper_mix_norm(xs, eps, h32=total, keep=False, **last)
+        assert torch.equal(before, xs)
+        want = sum(ref)
+        assert (total.double().cpu() - want).abs().max().item() < 1e-5 * max(1.0, want.abs().max().item())
+
+
+@pytest.mark.gpu
+@pytest.mark.parametrize("taps,W", [(1, 40), (2, 37), (3, 256), (4, 1000), (4, 2048)])
+def test_single_rows_convolve_in_the_boundary_kernel(taps, W):
+    """steps of one row per request on scattered slots that hold NaNs: equal, slot and output, to the same boundary followed by
+    the convolution kernel, and right from a sequence's first token on"""
+    from vox_serve_b200 import ops
+
+    g = torch.Generator().manual_seed(taps)
+    r = lambda *s: torch.randn(*s, generator=g, dtype=F32)
+    S, n, lens = 2, 6, 9
+    slots = torch.tensor([4, 0, 7, 2, 5, 1], dtype=I32, device=DEV)
+    cw, w, a = r(W, taps), r(W), r(S)
+    xs_in = [r(n, W) for _ in range(lens)]
+    mk_state = lambda: torch.full((8, max(taps - 1, 1), W), float("nan"), dtype=F32, device=DEV)
+    st1, st2 = mk_state(), mk_state()
+    h_ref = [O.rms_norm(O.read_streams([x.double()] * S, a.double()), w.double(), 1e-5) for x in xs_in]
+    for t in range(lens):
+        pos = torch.full((n,), t, dtype=I32, device=DEV)
+        qo = torch.arange(n + 1, dtype=I32, device=DEV)
+        rr = torch.arange(n, dtype=I32, device=DEV)
+        x0 = xs_in[t].to(DEV)
+        args = dict(x0=x0, in_c=a.to(DEV), w=w.to(DEV))
+        for dt in (BF16, F32):                      # (the second call starts from the state the first one left: put it back)
+            keep = st1.clone()
+            got = torch.zeros(n, W, dtype=dt, device=DEV)
+            ops.hyper_mix_norm(torch.zeros(n, S, W, device=DEV), 1e-5, h=got, conv=(cw.to(DEV).contiguous(), st1, pos, slots), **args)
+            if dt == BF16:
+                st1 = keep
+        h32 = torch.zeros(n, W, dtype=F32, device=DEV)
+        two = torch.zeros(n, W, dtype=F32, device=DEV)
+        ops.hyper_mix_norm(torch.zeros(n, S, W, device=DEV), 1e-5, h32=h32, **args)
+        ops.short_conv(h32, cw.to(DEV).contiguous(), None, st2, qo, rr, pos, slots, n, out=two, residual=True)
+        assert torch.equal(got, two), t
+        if taps > 1:
+            assert torch.equal(st1.nan_to_num(nan=7.0), st2.nan_to_num(nan=7.0)), t
+        want = h_ref[t].clone()
+        for j in range(taps):
+            if t - taps + 1 + j >= 0:
+                want += cw[:, j].double() * h_ref[t - taps + 1 + j]
+        assert (got.double().cpu() - want).abs().max().item() < 1e-5 * max(1.0, want.abs().max().item()), t
+
+
+@pytest.mark.gpu
+@pytest.mark.parametrize("dtype", [F32, BF16])
+@pytest.mark.parametrize("H,G,D,V,dims", [(4, 2, 12, 6, 8), (6, 6, 5, 3, 4), (8, 1, 64, 48, 64), (3, 3, 7, 1, 0)])
+def test_projection_tail_biases_rotation_values_and_factors(dtype, H, G, D, V, dims):
+    """the tail of an attention projection against the oracle's pieces: the bias enters before the rotation and before the value
+    norm, the head's factor reaches queries only, and portions of two requests land on their own pages at their own positions"""
+    from vox_serve_b200 import ops
+    from vox_serve_b200.hybrid_engine import RotaryConfig
+
+    g = torch.Generator().manual_seed(H + D)
+    r = lambda *s: torch.randn(*s, generator=g, dtype=F32)
+    lens, page, eps = [21, 6], 4, 1e-3
+    indptr, pages, n_pages = _paged(lens, page, seed=2)
+    P = H * D + G * D + G * V
+    rows, bias, fac = [r(n, P + 3) for n in lens], r(P), r(H)
+    rot = {"dims": dims, "base": 50.0, "scaling": {"factor": 3.0}}
+    kc = torch.full((n_pages, page, G, D), float("nan"), dtype=dtype, device=DEV)
+    vc = torch.full((n_pages, page, G, V), float("nan"), dtype=dtype, device=DEV)
+    q_all = [[], []]
+    for spans in ([(0, 9), (0, 1)], [(9, 1), (1, 5)], [(10, 11), (6, 0)]):
+        qo, row_req, pos = _step_tables(spans)
+        proj = torch.cat([rows[b][p0:p0 + n] for b, (p0, n) in enumerate(spans)], 0).to(DEV).contiguous()
+        T = proj.shape[0]
+        cs = None
+        if dims:
+            f = RotaryConfig(dims, 50.0, 3.0, layout="half", scaling="linear").frequencies().to(DEV)
+            cs = ops.rotary_table(pos, f, torch.zeros(T, 2, dims // 2, dtype=F32, device=DEV))
+        q = torch.zeros(T, H * D, dtype=dtype, device=DEV)
+        ops.qkv_norm_rotary_append(proj, 0, H * D, H * D + G * D, cs, dims // 2, "half", None, None, eps, q, kc, vc, row_req, pos, indptr,
+                                   pages, T, H, bias=bias.to(DEV), q_scale=fac.to(DEV), v_norm=True)
+        for b, (_, n) in enumerate(spans):
+            q_all[b].append(q[int(qo[b]):int(qo[b]) + n].double().cpu())
+    tol = 2e-5 if dtype == F32 else 4e-2
+    for b, n in enumerate(lens):
+        z = rows[b][:, :P].double() + bias.double()
+        q0, k0, v0 = z[:, :H * D].view(n, H, D), z[:, H * D:(H + G) * D].view(n, G, D), z[:, (H + G) * D:].view(n, G, V)
+        if dims:
+            q0, k0 = O.rotate_halves(q0, list(range(n)), rot), O.rotate_halves(k0, list(range(n)), rot)
+        q0 = q0 * fac.double().view(1, H, 1)
+        assert (torch.cat(q_all[b], 0).view(n, H, D) - q0).abs().max().item() < tol * max(1.0, q0.abs().max().item())
+        assert (_gather(kc, indptr, pages, b, n) - k0).abs().max().item() < tol * max(1.0, k0.abs().max().item())
+        assert (_gather(vc, indptr, pages, b, n) - O.unit_rms(v0, eps)).abs().max().item() < tol * 2
+
+
+@pytest.mark.gpu
+@pytest.mark.parametrize("dtype", [F32, BF16])
+@pytest.mark.parametrize("Q,R,Rd,dims", [(20, 12, 6, 6), (96, 64, 16, 8), (5, 3, 1, 0), (33, 40, 0, 0)])
+def test_latent_rows_and_query_latent(dtype, Q, R, Rd, dims):
+    from vox_serve_b200 import ops
+    from vox_serve_b200.hybrid_engine import RotaryConfig
+
+    g = torch.Generator().manual_seed(Q)
+    r = lambda *s: torch.randn(*s, generator=g, dtype=F32)
+    n, page, eps = 19, 4, 1e-2
+    indptr, pages, n_pages = _paged([n], page, seed=4)
+    rows, wq, wc = r(n, Q + R + Rd + 5), r(Q), r(R)
+    cache = torch.full((n_pages, page, 1, R + Rd), float("nan"), dtype=dtype, device=DEV)
+    cq_all = []
+    for p0, m in ((0, 1), (1, 7), (8, 11)):
+        qo, row_req, pos = _step_tables([(p0, m)])
+        cs = None
+        if dims:
+            f = RotaryConfig(dims, 30.0, layout="half", scaling="linear").frequencies().to(DEV)
+            cs = ops.rotary_table(pos, f, torch.zeros(m, 2, dims // 2, dtype=F32, device=DEV))
+        cq = torch.zeros(m, Q, dtype=dtype, device=DEV)
+        ops.latent_norm_append(rows[p0:p0 + m].to(DEV).contiguous(), 0, Q, Q, R, wq.to(DEV), wc.to(DEV), cq, cache, row_req, pos, indptr,
+                               pages, m, eps, rot=Rd, cs=cs, half=dims // 2, layout="half")
+        cq_all.append(cq.double().cpu())
+    z = rows.double()
+    kr = z[:, Q + R:Q + R + Rd]
+    if dims:
+        kr = O.rotate_halves(kr, list(range(n)), {"dims": dims, "base": 30.0})
+    want = torch.cat([O.rms_norm(z[:, Q:Q + R], wc.double(), eps), kr], 1)
+    tol = 2e-5 if dtype == F32 else 4e-2
+    assert (torch.cat(cq_all, 0) - O.rms_norm(z[:, :Q], wq.double(), eps)).abs().max().item() < tol * 2
+    assert (_gather(cache, indptr, pages, 0, n)[:, 0] - want).abs().max().item() < tol * max(1.0, want.abs().max().item())
+
+
+def _attend(q, k, v, dtype, page, window, scale, sink, mode, seed=6, lens=None):
+    """one or several sequences through the attention kernels: "tiles" (prompt portions), "rows" (single rows, keys split over
+    CTAs where there are few), "heads" (single rows as tiles over the heads).  q [T, H, D] float64 in the operand type's values."""
+    from vox_serve_b200 import ops
+
+    lens = lens or [q.shape[0]]
+    T, H, D = q.shape
+    G, V = k.shape[1], v.shape[2]
+    indptr, pages, n_pages = _paged(lens, page, seed=seed)
+    kc = torch.zeros(n_pages, page, G, D, dtype=dtype, device=DEV)
+    vc = torch.zeros(n_pages, page, G, V, dtype=dtype, device=DEV)
+    t0 = 0
+    for b, n in enumerate(lens):
+        pg = pages[int(indptr[b]):int(indptr[b + 1])].tolist()
+        for t in range(n):
+            kc[pg[t // page], t % page], vc[pg[t // page], t % page] = k[t0 + t].to(dtype), v[t0 + t].to(dtype)
+        t0 += n
+    qo, row_req, pos = _step_tables([(0, n) for n in lens])
+    out = torch.zeros(T, H * V, dtype=dtype, device=DEV)
+    qd = q.reshape(T, -1).to(dtype).to(DEV).contiguous()
+    sk = sink.to(F32).to(DEV) if sink is not None else None
+    args = (qd, kc, vc, out, None, row_req, pos, indptr, pages, T, H, G, D, V, window, scale)
+    if mode == "tiles":
+        R = ops.window_attn_tile_rows()
+        tl = [(b, r) for b, n in enumerate(lens) for r in range(int(qo[b]), int(qo[b]) + n, R)]
+        ops.window_attn(*args, tiles=(qo, torch.tensor([b for b, _ in tl], dtype=I32, device=DEV),
+                                      torch.tensor([r for _, r in tl], dtype=I32, device=DEV), len(tl)), sink=sk)
+    else:
+        # a few rows at a time: their keys are dealt to several CTAs and merged
+        scratch = torch.zeros(256 * 8 * H * (V + 2), dtype=F32, device=DEV)
+        for r0 in range(0, T, 16):
+            idx = torch.arange(r0, min(r0 + 16, T), dtype=I32, device=DEV)
+            ops.window_attn(*args, scratch=scratch, rows=(idx, idx.numel()), head_rows=mode == "heads", sink=sk)
+        o2 = torch.zeros_like(out)
+        ops.window_attn(*args[:3], o2, *args[4:], head_rows=mode == "heads", sink=sk)          # and all at once, unsplit
+        assert (o2.double() - out.double()).abs().max().item() < (1e-5 if dtype == F32 else 3e-2)
+    return out.double().cpu().view(T, H, V)
+
+
+@pytest.mark.gpu
+@pytest.mark.parametrize("mode", ["tiles", "rows", "heads"])
+@pytest.mark.parametrize("dtype,H,G,D,V", [(F32, 4, 2, 12, 6), (BF16, 8, 2, 64, 32), (BF16, 6, 1, 16, 128), (F32, 34, 2, 8, 5),
+                                           (BF16, 3, 3, 10, 7)])
+def test_sink_takes_the_weight_that_no_key_earns(mode, dtype, H, G, D, V):
+    """Scores of single keys are made to stand out, upwards and downwards: rows whose keys all score far below the sink give
+    (almost) nothing, rows that see the one hot key, hundreds of positions and dozens of pages away, give its value, rows of scores
+    near zero are divided by one more than their keys; sinks other than zero, per head; a request of one token beside it."""
+    g = torch.Generator().manual_seed(H * D)
+    lens, T = [200, 1, 67], 268
+    q = torch.randn(T, H, D, generator=g, dtype=F64) * 0.05
+    k = torch.randn(T, G, D, generator=g, dtype=F64) * 0.05
+    v = torch.randn(T, G, V, generator=g, dtype=F64)
+    q[:, :, 0] = 3.0
+    k[3, :, 0] = 5.0                                    # request 0: hot from position 3 on (score ~ 15 against ~ 0)
+    k[200:, :, 0] = -6.0                                # request 1 and the start of request 2: every score ~ -18: the sink wins
+    k[200 + 1 + 30, :, 0] = 4.0                         # request 2: a hot key at position 30
+    q, k, v = (t.to(dtype).to(F64) for t in (q, k, v))
+    tol = 2e-5 if dtype == F32 else 4e-2
+    for sink in (torch.zeros(H, dtype=F64), torch.linspace(-4.0, 6.0, H, dtype=F64), None):
+        ref, t0 = [], 0
+        for n in lens:
+            o = torch.zeros(n, H, V, dtype=F64)
+            for h in range(H):
+                s = (q[t0:t0 + n, h] @ k[t0:t0 + n, h // (H // G)].T)
+                s = torch.where(O.visible(n, 0), s, torch.full_like(s, -1e30))
+                if sink is None:
+                    p = torch.softmax(s, -1)
+                else:
+                    p = torch.softmax(torch.cat([s, sink[h].view(1, 1).expand(n, 1)], 1), -1)[:, :n]
+                o[:, h] = p @ v[t0:t0 + n, h // (H // G)]
+            ref.append(o)
+            t0 += n
+        ref = torch.cat(ref, 0)
+        if sink is not None and float(sink.abs().max()) == 0.0:
+            own = torch.cat([O.attend(q[a:a + n], k[a:a + n], v[a:a + n], 1.0, 0, True) for a, n in ((0, 200), (200, 1), (201, 67))], 0)
+            assert (own - ref).abs().max().item() < 1e-12
+            assert ref[200].abs().max() < 1e-5 and ref[201:231].abs().max() < 1e-5          # nothing but the sink
+            assert (ref[199] - v[3].repeat_interleave(H // G, 0)).abs().max() < 0.05         # the far key
+        got = _attend(q, k, v, dtype, 8, 0, 1.0, sink, mode, lens=lens)
+        assert (got - ref).abs().max().item() < tol * max(1.0, ref.abs().max().item()), sink
+
+
+@pytest.mark.gpu
+@pytest.mark.parametrize("mode", ["tiles", "rows", "heads"])
+@pytest.mark.parametrize("dtype", [F32, BF16])
+@pytest.mark.parametrize("window,page", [(1, 8), (7, 8), (64, 16), (65, 8), (100, 8)])
+def test_window_edges_with_a_sink(mode, dtype, window, page):
+    """hot keys at both ends of a page, of a tile of 64 rows and of the sequence are seen to distance window - 1 and by nothing
+    further; behind them only the sink is left (all other scores lie far below it)"""
+    H, G, D, V, T = 4, 2, 16, 16, 230
+    g = torch.Generator().manual_seed(window)
+    q, k = torch.randn(T, H, D, generator=g, dtype=F64) * 0.05, torch.randn(T, G, D, generator=g, dtype=F64) * 0.05
+    v = torch.randn(T, G, V, generator=g, dtype=F64)
+    q[:, :, 1], k[:, :, 1] = 4.0, -5.0
+    hots = [0, 1, 63, 64, 127, 128, T - 1]
+    k[hots, :, 1] = 4.0
+    q, k, v = (t.to(dtype).to(F64) for t in (q, k, v))
+    ref = O.attend(q, k, v, 1.0, window, True)
+    for hp in (64, 128):
+        if hp + window < T and not any(hp < o <= hp + window for o in hots):
+            assert ref[hp + window - 1].abs().max() > 0.3 and ref[hp + window].abs().max() < 1e-3
+    got = _attend(q, k, v, dtype, page, window, 1.0, torch.zeros(H, dtype=F64), mode)
+    assert (got - ref).abs().max().item() < (2e-5 if dtype == F32 else 4e-2)
+
+
+@pytest.mark.gpu
+@pytest.mark.parametrize("kind", ["latent", "attn"])
+def test_far_and_edge_tokens_show_in_a_models_logits(kind):
+    """One token id gets a key that every query scores high: decoded and prompt positions just inside and just outside its window
+    (latent attention), or hundreds of tokens away (attention), differ from a sequence without that token exactly where the
+    oracle's do."""
+    cfg = O.make_config(layers=(kind + "-",), loop=None, canon=0, l_window=24, width=64, a_rot_dims=0, l_rot=0, l_heads=2, a_heads=2)
+    sd = O.make_weights(cfg, 41)
+    hot_id, T = 96, 150
+    sd["embed"][:, 0] = 0.0
+    sd["embed"][:, 1] = 1.0
+    sd["embed"][hot_id, 0] = 40.0
+    if kind == "attn":
+        sd["l0.mix.k"][:, 0], sd["l0.mix.q"][:, 1] = 3.0, 3.0
+    else:
+        sd["l0.mix.dkv"][:, 0], sd["l0.mix.uk"][:] = 1.0, sd["l0.mix.uk"].abs()
+        sd["l0.mix.dq"][:, 1], sd["l0.mix.uq"][:] = 2.0, sd["l0.mix.uq"].abs()
+    base = [t % 90 for t in _tokens(T, 90, 8)]
+    at = 40
+    with_hot = base[:at] + [hot_id] + base[at + 1:]
+    ref = {n: O.forward(cfg, sd, t) for n, t in (("b", base), ("h", with_hot))}
+    diff = (ref["h"] - ref["b"]).abs().max(-1).values
+    if kind == "latent":
+        assert diff[at + 23] > 1e-2 and diff[at + 24:].max() < 1e-9
+    else:
+        assert diff[T - 1] > 1e-2
+    w = _worker(cfg, sd, F32, pages=60)
+    for steps in ([[("h", T)]], [[("h", 50)]] + [[("h", 1)]] * 100, [[("h", 63)], [("h", 1)], [("h", 2)], [("h", 84)]]):
+        got = _replay(w, {"h": with_hot}, steps)["h"]
+        assert _err(got, ref["h"]) < TOL[F32]
+        d = (got.double() - ref["b"]).abs().max(-1).values
+        assert ((d > 5e-3) == (diff > 5e-3)).all()
+
+
+@pytest.mark.gpu
+@pytest.mark.parametrize("T,W,ff", [(5, 64, 48), (130, 128, 200), (300, 48, 33), (17, 37, 20)])
+def test_gated_gelu_epilogues(T, W, ff):
+    from vox_serve_b200 import ops
+
+    g = torch.Generator().manual_seed(T)
+    h, gw, uw = (torch.randn(*s, generator=g) for s in ((T, W), (ff, W), (ff, W)))
+    for dt in (F32, BF16):
+        hd, gd, ud = (t.to(dt).to(DEV) for t in (h, gw * 0.3, uw * 0.3))
+        want = O.gelu_tanh(hd.double() @ gd.double().T) * (hd.double() @ ud.double().T)
+        tol = (1e-5 if dt == F32 else 1e-2) * max(1.0, want.abs().max().item())
+        out = torch.zeros(T, ff, dtype=dt, device=DEV)
+        ops.linear(hd, torch.cat([gd, ud], 0).contiguous(), out, epilogue=5)
+        assert (out.double() - want).abs().max().item() < tol
+        if dt == BF16 and W % 8 == 0:
+            half = ops.gate_up_tile_half(ff)
+            pw = ops.pack_weight(ops.interleave_gate_up(gd.contiguous(), ud.contiguous(), half), 2 * half)
+            out2 = torch.zeros(T, ff, dtype=dt, device=DEV)
+            ops.gemm(hd.contiguous(), pw, mode=2, out=out2, tile_rows=pw.tile_rows, n_out=ff, act="gelu_tanh")
+            assert (out2.double() - want).abs().max().item() < tol
+
+
+# ---- serving ---------------------------------------------------------------------------------------------------------
+@pytest.mark.gpu
+@pytest.mark.parametrize("dtype", [F32, BF16])
+def test_greedy_generation_through_scheduler(dtype):
+    """ModelWorker + Scheduler: three requests of unequal prompts, prompts fed in portions of 16 beside decoding requests,
+    more requests than slots.  Tokens equal the oracle's greedy tokens wherever the oracle's top-2 margin is clear."""
+    from vox_serve_b200.requests import Request
+    from vox_serve_b200.sampling import SamplingConfig
+    from vox_serve_b200.scheduler import Scheduler
+
+    cfg = O.make_config(layers=("latent", "attn", "latent-", "attn-"), loop=(1, 3, 2))
+    sd = O.make_weights(cfg, 13)
+    prompts = {"r0": _tokens(41, cfg["vocab"], 1), "r1": _tokens(5, cfg["vocab"], 2), "r2": _tokens(23, cfg["vocab"], 3)}
+    n_new = 12
+    w = _worker(cfg, sd, dtype, slots=2, pages=40, page_size=8)
+    sch = Scheduler(w, prefill_chunk_tokens=16)
+    reqs = {}
+    for rid, p in prompts.items():
+        reqs[rid] = Request(request_id=rid, prompt=p, sampling_config=SamplingConfig(greedy=True, max_tokens=n_new))
+        sch.submit(reqs[rid])
+    sch.run_until_done(max_steps=400)
+    assert len(sch.finished) == 3 and w.empty_pages.qsize() == 40 and len(w.free_slots) == 2
+    margin = 0.05 if dtype == F32 else 0.25
+    wrong = clear = 0
+    for rid, p in prompts.items():
+        got = [int.from_bytes(c, "little", signed=True) for c in sch.audio[rid]]
+        assert len(got) == n_new and reqs[rid].finish_reason == "max_tokens_reached"
+        toks = list(p)
+        for t in got:                       # teacher-forced comparison: every step is judged on the framework's own prefix
+            z = O.forward(cfg, sd, toks)[-1]
+            top = torch.topk(z, 2)
+            if float(top.values[0] - top.values[1]) > margin:
+                clear += 1
+                wrong += t != int(top.indices[0])
+            toks.append(t)
+    assert wrong == 0 and clear > n_new, (wrong, clear)
+
+
+def _write_model_dir(d, cfg, sd):
+    """config.json + model.safetensors (8-byte length, JSON header, raw little-endian data) of a bfloat16 checkpoint"""
+    import struct
+
+    meta, blobs, off = {}, [], 0
+    for k, v in sd.items():
+        raw = v.contiguous().reshape(-1).view(torch.uint8).numpy().tobytes()
+        meta[k] = {"dtype": "BF16", "shape": list(v.shape), "data_offsets": [off, off + len(raw)]}
+        blobs.append(raw)
+        off += len(raw)
+    head = json.dumps(meta).encode()
+    with open(os.path.join(d, "model.safetensors"), "wb") as f:
+        f.write(struct.pack("<Q", len(head)) + head + b"".join(blobs))
+    with open(os.path.join(d, "config.json"), "w") as f:
+        json.dump(cfg, f)
+
+
+@pytest.mark.gpu
+def test_command_lines_on_a_model_directory(capsys):
+    """a checkpoint directory through the trace replay tool (a subprocess: portions, two requests, a request ended and its
+    slot taken again) and through the generate command (in process)."""
+    import subprocess
+    import sys
+
+    import numpy as np
+
+    from vox_serve_b200 import generate
+
+    root = os.path.dirname(os.path.dirname(os.path.abspath(__file__)))
+    cfg = O.make_config(layers=("latent", "attn", "latent-", "attn-"), loop=(1, 3, 2))
+    sd = O.make_weights(cfg, 17)
+    V = cfg["vocab"]
+    a, b, c = _tokens(30, V, 1), _tokens(12, V, 2), _tokens(9, V, 3)
+    with tempfile.TemporaryDirectory() as d:
+        _write_model_dir(d, cfg, sd)
+        out = os.path.join(d, "out")
+        steps = [{"step": 0, "entries": [{"id": "a", "tokens": a[:20], "want": [0, 19]}, {"id": "b", "tokens": b[:2], "want": []}], "end": []},
+                 {"step": 1, "entries": [{"id": "a", "tokens": a[20:21], "want": [0]}, {"id": "b", "tokens": b[2:], "want": [9]}], "end": ["b"]},
+                 {"step": 2, "entries": [{"id": "c", "tokens": c, "want": [8]}, {"id": "a", "tokens": a[21:], "want": [8]}], "end": ["a", "c"]}]
+        r = subprocess.run([sys.executable, os.path.join(root, "bin", "trace_run"), "--model", d, "--dtype", "float32", "--out", out,
+                            "--max-tokens", "128"], input="".join(json.dumps(s) + "\n" for s in steps), capture_output=True,
+                           text=True, timeout=900)
+        assert r.returncode == 0, r.stderr[-2000:]
+        assert [ln for ln in r.stdout.splitlines() if ln.startswith("done")] == ["done 0", "done 1", "done 2"]
+        ra, rb, rc = (O.forward(cfg, sd, t) for t in (a, b, c))
+        want = {0: torch.stack([ra[0], ra[19]]), 1: torch.stack([ra[20], rb[11]]), 2: torch.stack([rc[8], ra[29]])}
+        for s_, ref in want.items():
+            got = torch.from_numpy(np.fromfile(os.path.join(out, f"{s_}.f32"), dtype="<f4").reshape(2, V).copy())
+            assert _err(got, ref) < TOL[F32], s_
+        capsys.readouterr()
+        assert generate.main(["--model", d, "--prompt", " ".join(map(str, a)), "--prompt", " ".join(map(str, b)), "--max-new", "6",
+                              "--dtype", "float32", "--prefill-chunk", "16", "--page-size", "8"]) == 0
+        lines = capsys.readouterr().out.strip().splitlines()[-2:]
+        for line, prompt in zip(lines, (a, b)):
+            toks = list(prompt)
+            for t in (int(x) for x in line.split()):
+                z = O.forward(cfg, sd, toks)[-1]
+                top = torch.topk(z, 2)
+                assert float(top.values[0] - top.values[1]) < 0.05 or t == int(top.indices[0])
+                toks.append(t)
+            assert len(toks) == len(prompt) + 6
