@@ -205,6 +205,7 @@ OTHER_SIZES = [
     dict(l_window=5, a_window=9, canon=6, streams=5, loop=(0, 4, 2), width=50, eps=1e-2),
     dict(l_heads=18, a_heads=34, a_kv_heads=2, a_dim=4, a_vdim=3, a_rot_dims=2, l_dim=4, l_rot=2, l_vdim=3, l_rank=24, l_q_rank=8, canon=4),
     dict(width=37, vocab=31, streams=2, canon=3, l_rank=11, l_rot=2, l_dim=1, l_vdim=1, a_dim=2, a_vdim=1, a_rot_dims=2),
+    dict(l_rank=256, l_rot=64, l_dim=128, l_vdim=128, l_q_rank=200, a_dim=256, a_vdim=256, a_rot_dims=64, a_heads=2, l_heads=2, streams=2),
     dict(a_base=12.0, a_factor=1.0, l_base=9.0, l_window=40, streams=7, canon=5, a_kv_heads=4),
 ]
 
@@ -213,7 +214,7 @@ OTHER_SIZES = [
 @pytest.mark.parametrize("kw", OTHER_SIZES)
 def test_other_sizes(kw):
     """head counts of one and many, key/value heads = heads and = 1, key size != value size, sizes of one and odd sizes that rule
-    tensor-core projections and 16-byte rows out, windows of one / none (on both mixers), no rotated part and rotation on a slice,
+    tensor-core projections and 16-byte rows out, the largest heads, windows of one / none (on both mixers), no rotated part and rotation on a slice,
     scaling by one and none, convolutions of no tap, one and more taps than the fused form takes, one to seven streams, loops of
     several spans, a large eps."""
     cfg = O.make_config(layers=("latent", "attn", "latent-", "attn-"), **{"loop": (1, 3, 2), **kw})

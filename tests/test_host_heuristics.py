@@ -131,3 +131,31 @@ def test_speech_tokenizer_config_and_mask_bounds():
         am[:, :valid] = 1
         assert torch.equal(GLMWhisperVQEncoder.block_causal_bounds(valid, T, block, "cpu"),
                            oenc.block_causal_bounds(am, block))
+
+
+def test_graph_capture_holds_the_garbage_collector_back(monkeypatch):
+    """a dead CUDA graph that the collector finds inside a capture would end it: no collection happens there, and the
+    collector's state is restored afterwards, also after an error"""
+    import gc
+    from contextlib import nullcontext
+
+    import torch
+
+    from vox_serve_b200.worker.base import capture_graph
+
+    monkeypatch.setattr(torch.cuda, "graph", lambda g, pool=None, stream=None: nullcontext())
+    was = gc.isenabled()
+    try:
+        for before in (True, False):
+            gc.enable() if before else gc.disable()
+            with capture_graph(None, None):
+                assert not gc.isenabled()
+            assert gc.isenabled() == before
+            try:
+                with capture_graph(None, None):
+                    raise KeyError
+            except KeyError:
+                pass
+            assert gc.isenabled() == before
+    finally:
+        gc.enable() if was else gc.disable()

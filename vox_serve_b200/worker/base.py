@@ -19,8 +19,10 @@ There is no CPU / eager fallback: a missing libvoxb200.so raises at construction
 """
 from __future__ import annotations
 
+import gc
 import os
 import queue
+from contextlib import contextmanager
 from typing import Coroutine, Dict, List, Optional
 
 import numpy as np
@@ -33,6 +35,21 @@ from ..model import load_model
 from ..requests import LMInputs, Request
 
 I32 = torch.int32
+
+
+@contextmanager
+def capture_graph(g: torch.cuda.CUDAGraph, stream: torch.cuda.Stream, pool=None):
+    """Captures the launches of the block into ``g``, with the cyclic garbage collector held back meanwhile: a collection that
+    happened to fall into the block could destroy a dead CUDA graph (of a worker that is gone), a call the runtime does not
+    permit while a stream captures and which invalidates this capture."""
+    collecting = gc.isenabled()
+    gc.disable()
+    try:
+        with torch.cuda.graph(g, pool=pool, stream=stream):
+            yield
+    finally:
+        if collecting:
+            gc.enable()
 
 
 class _Staging:
@@ -250,7 +267,7 @@ class ModelWorker:
         ds.wait_stream(torch.cuda.current_stream())
         before = ops.launch_count()
         with torch.cuda.stream(ds):
-            with torch.cuda.graph(g, pool=self.voc_pool, stream=ds):
+            with capture_graph(g, ds, self.voc_pool):
                 self._vocoder_body(n)
         torch.cuda.current_stream().wait_stream(ds)
         if self.voc_pool is None:
@@ -472,7 +489,7 @@ class ModelWorker:
         s.wait_stream(torch.cuda.current_stream())
         before = ops.launch_count()
         with torch.cuda.stream(s):
-            with torch.cuda.graph(g, pool=self.graph_pool, stream=s):
+            with capture_graph(g, s, self.graph_pool):
                 self._device_step(B, B, False)
         torch.cuda.current_stream().wait_stream(s)
         if self.graph_pool is None:
@@ -619,7 +636,7 @@ class ModelWorker:
                 s.wait_stream(torch.cuda.current_stream())
                 before = ops.launch_count()
                 with torch.cuda.stream(s):
-                    with torch.cuda.graph(g, pool=self.graph_pool, stream=s):
+                    with capture_graph(g, s, self.graph_pool):
                         fn()
                 torch.cuda.current_stream().wait_stream(s)
                 if self.graph_pool is None:
