@@ -205,7 +205,8 @@ OTHER_SIZES = [
     dict(l_window=5, a_window=9, canon=6, streams=5, loop=(0, 4, 2), width=50, eps=1e-2),
     dict(l_heads=18, a_heads=34, a_kv_heads=2, a_dim=4, a_vdim=3, a_rot_dims=2, l_dim=4, l_rot=2, l_vdim=3, l_rank=24, l_q_rank=8, canon=4),
     dict(width=37, vocab=31, streams=2, canon=3, l_rank=11, l_rot=2, l_dim=1, l_vdim=1, a_dim=2, a_vdim=1, a_rot_dims=2),
-    dict(l_rank=256, l_rot=64, l_dim=128, l_vdim=128, l_q_rank=200, a_dim=256, a_vdim=256, a_rot_dims=64, a_heads=2, l_heads=2, streams=2),
+    dict(l_rank=256, l_rot=64, l_dim=128, l_vdim=128, l_q_rank=200, a_dim=256, a_vdim=256, a_rot_dims=64, a_heads=2, l_heads=2,
+         streams=2, l_scale=0.05, a_scale=0.06),
     dict(a_base=12.0, a_factor=1.0, l_base=9.0, l_window=40, streams=7, canon=5, a_kv_heads=4),
 ]
 
@@ -420,6 +421,40 @@ def test_single_rows_convolve_in_the_boundary_kernel(taps, W):
             if t - taps + 1 + j >= 0:
                 want += cw[:, j].double() * h_ref[t - taps + 1 + j]
         assert (got.double().cpu() - want).abs().max().item() < 1e-5 * max(1.0, want.abs().max().item()), t
+
+
+@pytest.mark.gpu
+@pytest.mark.parametrize("taps,C,act,res", [(2, 64, None, True), (3, 520, "silu", False), (4, 1028, None, True), (4, 12, "silu", True)])
+def test_convolution_of_long_steps_in_16_byte_pieces(taps, C, act, res):
+    """prompt portions of four requests (one of them a single row) in steps of 64 rows and more, cut so that requests begin and end
+    at every place of a group of rows, on slots that hold NaNs"""
+    from vox_serve_b200 import ops
+
+    g = torch.Generator().manual_seed(C)
+    w, bv = torch.randn(C, taps, generator=g), torch.randn(C, generator=g)
+    lens = [131, 2, 96, 45]
+    xs = [torch.randn(n, C, generator=g) for n in lens]
+    for cuts in ([1000], [66, 1000], [29, 1, 1000], [67, 2, 3, 1000]):
+        state = torch.full((6, taps - 1, C), float("nan"), dtype=F32, device=DEV)
+        slots = torch.tensor([5, 1, 3, 0], dtype=I32, device=DEV)
+        at, outs = [0] * 4, [[] for _ in lens]
+        for c in cuts:
+            live = [(b, min(c, lens[b] - at[b])) for b in range(4) if at[b] < lens[b]]
+            qo, row_req, pos = _step_tables([(at[b], n) for b, n in live])
+            T = int(qo[-1])
+            x = torch.cat([xs[b][at[b]:at[b] + n] for b, n in live], 0).to(DEV)
+            o16, o32 = torch.zeros(T, C, dtype=BF16, device=DEV), torch.zeros(T, C + 4, dtype=F32, device=DEV)
+            ops.short_conv(x, w.to(DEV), bv.to(DEV), state, qo, row_req, pos, slots[[b for b, _ in live]].contiguous(), len(live), out=o16,
+                           out_f32=o32[:, :C], act=act, residual=res)
+            assert (o32[:, C:] == 0).all() and torch.equal(o16, o32[:, :C].to(BF16))
+            for i, (b, n) in enumerate(live):
+                outs[b].append(o32[int(qo[i]):int(qo[i]) + n, :C].double().cpu())
+                at[b] += n
+        for b in range(4):
+            r = O.causal_conv(xs[b].double(), w.double()) + bv.double()
+            r = r * O.sigmoid(r) if act else r
+            r = r + xs[b].double() if res else r
+            assert (torch.cat(outs[b], 0) - r).abs().max().item() < 1e-5 * max(1.0, r.abs().max().item()), (cuts, b)
 
 
 @pytest.mark.gpu

@@ -219,12 +219,12 @@ def forward(cfg: Dict[str, Any], sd: Dict[str, torch.Tensor], tokens: List[int],
 def make_config(layers=("latent", "attn", "latent-", "attn", "attn-"), width=48, vocab=97, eps=1e-5, streams=2, canon=3,
                 loop=(1, 3, 3), l_heads=3, l_dim=8, l_rot=6, l_rot_dims=None, l_vdim=10, l_rank=12, l_q_rank=20, l_window=11,
                 l_base=300.0, a_heads=4, a_kv_heads=2, a_dim=12, a_vdim=6, a_rot_dims=8, a_base=500.0, a_factor=4.0, a_window=0,
-                ff=40) -> Dict[str, Any]:
+                l_scale=0.27, a_scale=0.33, ff=40) -> Dict[str, Any]:
     """layers: "latent" or "attn"; a trailing "-" leaves the feed-forward out."""
     out = []
     for spec in layers:
         if spec.startswith("attn"):
-            m = {"heads": a_heads, "kv_heads": a_kv_heads, "dim": a_dim, "vdim": a_vdim, "scale": 0.33}
+            m = {"heads": a_heads, "kv_heads": a_kv_heads, "dim": a_dim, "vdim": a_vdim, "scale": a_scale}
             if a_rot_dims:
                 m["rot"] = {"base": a_base, "dims": a_rot_dims}
                 if a_factor:
@@ -233,7 +233,8 @@ def make_config(layers=("latent", "attn", "latent-", "attn", "attn-"), width=48,
                 m["mask"] = {"size": a_window}
             layer = {"type": "attention", "mixer": m}
         else:
-            m = {"heads": l_heads, "dim": l_dim, "rot_dim": l_rot, "vdim": l_vdim, "kv_rank": l_rank, "q_rank": l_q_rank, "scale": 0.27}
+            m = {"heads": l_heads, "dim": l_dim, "rot_dim": l_rot, "vdim": l_vdim, "kv_rank": l_rank, "q_rank": l_q_rank,
+                 "scale": l_scale}
             if l_window:
                 m["mask"] = {"size": l_window}
             if l_rot:

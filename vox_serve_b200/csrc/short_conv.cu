@@ -126,6 +126,81 @@ __global__ void __launch_bounds__(256) short_conv_rows_kernel(ShortConvParams p)
   }
 }
 
+// The same for rows that move in 16-byte pieces: a thread computes SC_VRPT consecutive rows of four neighbouring channels.  Row
+// groups that lie inside one request, past the reach of its slot -- nearly all of a long prompt -- take every input from the
+// rows and check nothing per row; the FMA chain of an output is that of the kernels above.
+constexpr int SC_VRPT = 4, SC_VTHREADS = 128;
+
+template <typename CT> __device__ __forceinline__ void sc_store4(CT* __restrict__ p, float a, float b, float c, float d);
+template <> __device__ __forceinline__ void sc_store4<float>(float* __restrict__ p, float a, float b, float c, float d) {
+  *reinterpret_cast<float4*>(p) = make_float4(a, b, c, d);
+}
+template <> __device__ __forceinline__ void sc_store4<__nv_bfloat16>(__nv_bfloat16* __restrict__ p, float a, float b, float c, float d) {
+  *reinterpret_cast<uint2*>(p) = make_uint2(pack_bf16(a, b), pack_bf16(c, d));
+}
+
+template <typename CT, int TAPS>
+__global__ void __launch_bounds__(SC_VTHREADS) short_conv_rows4_kernel(ShortConvParams p) {
+  constexpr int K = TAPS - 1;
+  const int c = (blockIdx.x * SC_VTHREADS + threadIdx.x) * 4, t0 = blockIdx.y * SC_VRPT;
+  if (c >= p.C) { pdl_sync(); return; }
+  float w[4][TAPS], bias[4];
+#pragma unroll
+  for (int e = 0; e < 4; ++e) {
+#pragma unroll
+    for (int j = 0; j < TAPS; ++j) w[e][j] = p.w[static_cast<size_t>(c + e) * TAPS + j];
+    bias[e] = p.bias ? p.bias[c + e] : 0.f;
+  }
+  pdl_sync();
+  float u[SC_VRPT + K][4];
+#pragma unroll
+  for (int i = 0; i < SC_VRPT + K; ++i) {
+    const int t = t0 - K + i;
+    float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
+    if (t >= 0 && t < p.T) v = *reinterpret_cast<const float4*>(p.in + static_cast<size_t>(t) * p.ld_in + c);
+    u[i][0] = v.x; u[i][1] = v.y; u[i][2] = v.z; u[i][3] = v.w;
+  }
+  const int b0 = p.row_req[t0];
+  const bool inside = t0 - p.qo_indptr[b0] >= K && p.row_req[min(t0 + SC_VRPT, p.T) - 1] == b0;
+#pragma unroll
+  for (int rr = 0; rr < SC_VRPT; ++rr) {
+    const int t = t0 + rr;
+    if (t >= p.T) break;
+    float h[K > 0 ? K : 1][4];                     // the inputs before the row's own, oldest first
+#pragma unroll
+    for (int j = 0; j < K; ++j)
+#pragma unroll
+      for (int e = 0; e < 4; ++e) h[j][e] = u[rr + j][e];
+    if (!inside) {
+      const int b = p.row_req[t], r = t - p.qo_indptr[b], ps = p.pos[t];
+      const float* st = p.state + (static_cast<size_t>(p.slots[b]) * K) * p.C + c;
+#pragma unroll
+      for (int j = 0; j < K; ++j) {
+        const int back = K - j;
+        if (ps - back < 0) {
+#pragma unroll
+          for (int e = 0; e < 4; ++e) h[j][e] = 0.f;
+        } else if (r - back < 0) {
+#pragma unroll
+          for (int e = 0; e < 4; ++e) h[j][e] = st[static_cast<size_t>(r + j) * p.C + e];
+        }
+      }
+    }
+    float acc[4];
+#pragma unroll
+    for (int e = 0; e < 4; ++e) {
+      acc[e] = bias[e];
+#pragma unroll
+      for (int j = 0; j < K; ++j) acc[e] = fmaf(w[e][j], h[j][e], acc[e]);
+      acc[e] = fmaf(w[e][K], u[rr + K][e], acc[e]);
+      if (p.act == 1) acc[e] = acc[e] / (1.f + expf(-acc[e]));
+      if (p.residual) acc[e] += u[rr + K][e];
+    }
+    if (p.out) sc_store4<CT>(static_cast<CT*>(p.out) + static_cast<size_t>(t) * p.ld_out + c, acc[0], acc[1], acc[2], acc[3]);
+    if (p.out_f32) sc_store4<float>(p.out_f32 + static_cast<size_t>(t) * p.ld_f32 + c, acc[0], acc[1], acc[2], acc[3]);
+  }
+}
+
 // the slot after the step: the last taps - 1 inputs of [old slot | the step's rows], zeros for positions before 0
 __global__ void __launch_bounds__(256) short_conv_state_kernel(ShortConvParams p) {
   pdl_sync();
@@ -221,7 +296,21 @@ int vb_short_conv(void* d_out, int ld_out, float* d_out_f32, int ld_f32, const f
   const int cx = (channels + 255) / 256;
   const dim3 rows_grid(cx, (T + SC_RPT - 1) / SC_RPT);
   const bool f32 = out_dtype == 1;
-  if (T >= 64 && taps == 2) {
+  auto fits = [](const void* q, int ld, size_t bytes) {
+    return q == nullptr || (ld % 4 == 0 && reinterpret_cast<uintptr_t>(q) % bytes == 0);
+  };
+  const bool vec = rows_form && channels % 4 == 0 && fits(d_in, ld_in, 16) && fits(d_out, ld_out, f32 ? 16 : 8) && fits(d_out_f32, ld_f32, 16);
+  const dim3 vec_grid((channels / 4 + SC_VTHREADS - 1) / SC_VTHREADS, (T + SC_VRPT - 1) / SC_VRPT);
+  if (vec && taps == 2) {
+    if (f32) VB_LAUNCH_PDL((short_conv_rows4_kernel<float, 2>), vec_grid, SC_VTHREADS, 0, stream, p);
+    else VB_LAUNCH_PDL((short_conv_rows4_kernel<bf16, 2>), vec_grid, SC_VTHREADS, 0, stream, p);
+  } else if (vec && taps == 3) {
+    if (f32) VB_LAUNCH_PDL((short_conv_rows4_kernel<float, 3>), vec_grid, SC_VTHREADS, 0, stream, p);
+    else VB_LAUNCH_PDL((short_conv_rows4_kernel<bf16, 3>), vec_grid, SC_VTHREADS, 0, stream, p);
+  } else if (vec && taps == 4) {
+    if (f32) VB_LAUNCH_PDL((short_conv_rows4_kernel<float, 4>), vec_grid, SC_VTHREADS, 0, stream, p);
+    else VB_LAUNCH_PDL((short_conv_rows4_kernel<bf16, 4>), vec_grid, SC_VTHREADS, 0, stream, p);
+  } else if (T >= 64 && taps == 2) {
     if (f32) VB_LAUNCH_PDL((short_conv_rows_kernel<float, 2>), rows_grid, 256, 0, stream, p);
     else VB_LAUNCH_PDL((short_conv_rows_kernel<bf16, 2>), rows_grid, 256, 0, stream, p);
   } else if (T >= 64 && taps == 3) {
