@@ -626,9 +626,11 @@ def main():
     ap.add_argument("--arch", default=None, choices=["bobavik", "razevik", "fovunex", "nadevik", "zopipel"],
                     help="instead of the headline workload: prefill / decode throughput of that design beside its closest "
                          "relative at equal size (bobavik: the Llama-shaped engine; razevik: Bobavik with attention layers "
-                         "only; fovunex, nadevik: Bobavik; zopipel: Fovunex and Bobavik; benchmarks/hybrid_bench.py); one JSON line per size")
+                         "only; fovunex, nadevik: Bobavik; zopipel: Fovunex and Bobavik; benchmarks/hybrid_bench.py); one JSON line "
+                         "per size")
     ap.add_argument("--arch-sizes", default="2048,3072", help="model widths of the --arch comparison")
-    ap.add_argument("--arch-only", default="", choices=["", "bobavik", "llama", "razevik", "fovunex", "nadevik", "zopipel"], help="run one side of the comparison")
+    ap.add_argument("--arch-only", default="", choices=["", "bobavik", "llama", "razevik", "fovunex", "nadevik", "zopipel"],
+                    help="run one side of the comparison")
     args = ap.parse_args()
     if args.arch is not None:
         from benchmarks import hybrid_bench

@@ -1,5 +1,6 @@
-"""Worker for text-only LMs on the hybrid engine (model/bobavik.py, model/razevik.py, model/fovunex.py, model/nadevik.py): the same five scheduler-facing methods, page pool,
-batch slots, packed staging buffer, sampled-id ring and decode CUDA graphs as ``ModelWorker``, with three differences.
+"""Worker for text-only LMs on the hybrid engine (model/bobavik.py, model/razevik.py, model/fovunex.py, model/nadevik.py,
+model/zopipel.py): the same five scheduler-facing methods, page pool, batch slots, packed staging buffer, sampled-id ring and
+decode CUDA graphs as ``ModelWorker``, with three differences.
 
   * Prompts are fed in portions.  A request carries ``pending_tokens`` (the rest of its prompt, or continuation tokens a
     client supplies); a step takes ``step_tokens`` of them (default: ``prefill_chunk_tokens``, or all), so portions of
