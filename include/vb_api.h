@@ -598,18 +598,22 @@ int vb_window_attn(void* d_out, const void* d_q, const void* d_k_cache, const vo
                    int ld_gate, const int32_t* d_row_req, const int32_t* d_pos, const int32_t* d_page_indptr,
                    const int32_t* d_page_indices, int T, int H, int G, int dim, int vdim, int page_size, int window,
                    float scale, int dtype, float* d_part, long long part_floats, const int32_t* d_row_list, int head_rows,
-                   int chunk, int k_ld, int v_ld, int v_share, int out_f32, const float* d_sink, void* stream);
+                   int chunk, int k_ld, int v_ld, int v_share, int out_f32, const float* d_sink, int keep_first,
+                   int head_gate, void* stream);
 /* (chunk > 0: a position sees only the keys of its own block of `chunk` positions, counted from position 0.  k_ld / v_ld:
  * elements per token of the key / value cache (<= 0: G * dim, (G / v_share) * vdim); a value that is a leading slice of
  * the single key head has v_ld = k_ld and the same base pointer.  v_share consecutive key heads read one value head.
  * out_f32: the output is fp32 [T][H * vdim] whatever the operand type.  d_sink [H] (optional): the denominator of head h's
- * softmax has exp(d_sink[h]) added, a further key of that score without a value.) */
+ * softmax has exp(d_sink[h]) added, a further key of that score without a value.  keep_first: positions 0 .. keep_first - 1
+ * are visible to every later position whatever the window or chunk says.  head_gate != 0: the gate row holds one value per
+ * head instead of one per output value.) */
 int vb_window_attn_tile_rows(void);
 int vb_window_attn_tiled(void* d_out, const void* d_q, const void* d_k_cache, const void* d_v_cache, const float* d_gate,
                          int ld_gate, const int32_t* d_pos, const int32_t* d_page_indptr, const int32_t* d_page_indices,
                          const int32_t* d_qo_indptr, const int32_t* d_tile_req, const int32_t* d_tile_row0, int n_tiles,
                          int T, int H, int G, int dim, int vdim, int page_size, int window, float scale, int dtype,
-                         int chunk, int k_ld, int v_ld, int v_share, int out_f32, const float* d_sink, void* stream);
+                         int chunk, int k_ld, int v_ld, int v_share, int out_f32, const float* d_sink, int keep_first,
+                   int head_gate, void* stream);
 /* Element-wise gated recurrence (minGRU) over fp32 state slots [slots][width]: z = sigmoid(pz + bz), u = px + bx,
  * c = u + 1/2 (u >= 0) or sigmoid(u), S_t = (1 - z) S_(t-1) + z c (S = 0 before position 0), out = S_t * silu(pg); pz, px,
  * pg are columns z_off, x_off, g_off of the fp32 projection rows.  single_rows / multi_rows select the requests served.
@@ -625,6 +629,35 @@ int vb_mingru_tiled(void* d_out, float* d_state, float* d_scratch, const float* 
                     const int32_t* d_slots, const int32_t* d_tile_req, const int32_t* d_tile_row0, int n_tiles, int tile_rows,
                     int B, int width, int out_dtype, void* stream);
 int vb_mingru_scratch_floats(int n_tiles, int tile_rows, int width);
+/* Real-gated linear recurrent unit over fp32 state slots [slots][width]: r = sigmoid(R_b u + br), i = sigmoid(I_b u + bi) in
+ * `blocks` equal parts of the channels (d_w [blocks][2 * bs][bs]: R_b above I_b, bf16 or fp32; d_bias [blocks][2 * bs]),
+ * log a = -c r softplus(d_lam), S_t = a S_(t-1) + sqrt(1 - a^2) i u, d_out = S * gelu_tanh(d_y + d_y_bias).  One launch serves
+ * requests that bring one row; multi_rows != 0: the others too, with d_ab fp32 [T][2][width], walked in order (n_tiles == 0)
+ * or in the tiles and pieces of vb_mingru_tiled (d_scratch: vb_mingru_scratch_floats floats). */
+int vb_rglru(void* d_out, int ld_out, float* d_state, float* d_ab, float* d_scratch, const float* d_u, int ld_u, const void* d_w,
+             const float* d_bias, const float* d_lam, float c, const float* d_y, int ld_y, const float* d_y_bias,
+             const int32_t* d_qo_indptr, const int32_t* d_row_req, const int32_t* d_pos, const int32_t* d_slots,
+             const int32_t* d_tile_req, const int32_t* d_tile_row0, int n_tiles, int tile_rows, int T, int B, int width,
+             int blocks, int multi_rows, int w_dtype, int out_dtype, void* stream);
+/* State-space duality (ssd.cu): per head an fp32 state [N][V] per slot, dt = softplus(d_dt + d_dt_bias),
+ * S_t = exp(-exp(A_log) dt) S_(t-1) + dt B_t x_t^T, y = S^T C + D x, d_out [T][H * V] = y * silu(d_z); d_xbc rows
+ * [x: H * V | B: G * N | C: G * N] in the compute type, head h reads group h / (H / G).  vb_ssd: row by row over the slot
+ * (single_rows / multi_rows select the requests).  vb_ssd_tiled: prompt portions in tiles of vb_ssd_tile_rows(V, N) rows (0:
+ * these sizes need vb_ssd), laid out as for vb_decay_attn_tiled; scratch: vb_ssd_scratch_floats floats.
+ * vb_group_rmsnorm: d_out (compute type) = rows of C channels in `groups` equal neighbourhoods, each divided by its own root
+ * mean square (eps inside the root), times d_w. */
+int vb_ssd(float* d_out, float* d_state, const void* d_xbc, int ld, const float* d_dt, int ld_dt, const float* d_dt_bias,
+           const float* d_A_log, const float* d_D, const float* d_z, int ld_z, const int32_t* d_qo_indptr, const int32_t* d_pos,
+           const int32_t* d_slots, int B, int H, int V, int N, int G, int single_rows, int multi_rows, int x_dtype,
+           void* stream);
+int vb_ssd_tile_rows(int V, int N);
+long long vb_ssd_scratch_floats(int n_tiles, int H, int V, int N);
+int vb_ssd_tiled(float* d_out, float* d_state, float* d_scratch, const void* d_xbc, int ld, const float* d_dt, int ld_dt,
+                 const float* d_dt_bias, const float* d_A_log, const float* d_D, const float* d_z, int ld_z,
+                 const int32_t* d_qo_indptr, const int32_t* d_pos, const int32_t* d_slots, const int32_t* d_tile_req,
+                 const int32_t* d_tile_row0, int n_tiles, int B, int H, int V, int N, int G, int x_dtype, void* stream);
+int vb_group_rmsnorm(void* d_out, const float* d_x, const float* d_w, int T, int C, int groups, float eps, int out_dtype,
+                     void* stream);
 /* Linear attention with a scalar decay per head; q, k, v = silu of the projection columns; state fp32
  * [slots][H][dim][vdim], zero for a request whose first new token has position 0.  single_rows / multi_rows select
  * the step kernel (requests bringing one token) and the chunked kernel (requests bringing more). */
@@ -656,6 +689,10 @@ int vb_moe_route_sigmoid(int32_t* d_idx, float* d_wts, float* d_shared_gate, con
 int vb_moe_route_groups(int32_t* d_idx, float* d_wts, float* d_shared_gate, const void* d_h, const float* d_router_w,
                         const float* d_correction, const float* d_shared_gate_w, int T, int width, int experts, int top,
                         int n_groups, int keep, int softmax_scores, int rank_by_max, int normalize, int h_dtype, void* stream);
+/* no scores: d_idx[t] = d_table[d_ids[t]] (int32 [vocab][top]), weights 1 / top; the shared gate as above */
+int vb_moe_route_table(int32_t* d_idx, float* d_wts, float* d_shared_gate, const int32_t* d_ids, const int32_t* d_table,
+                       const void* d_h, const float* d_shared_gate_w, int T, int width, int vocab, int experts, int top,
+                       int h_dtype, void* stream);
 int vb_moe_group(int32_t* d_row_off, int32_t* d_sorted_token, int32_t* d_pair_row, const int32_t* d_idx, int T,
                  int experts, int top, int tile_rows, int32_t* d_tile_group, int n_tiles, void* stream);
 /* (tile_rows > 0: every expert's rows start at a multiple of tile_rows; padding rows get token -1; d_tile_group[i] =
@@ -682,7 +719,8 @@ int vb_moe_combine(float* d_y, const float* d_expert_out, const float* d_shared_
  * vb_short_conv: causal convolution over time per channel of the fp32 columns d_in[t][0 .. channels), weights fp32
  *   [channels][taps] (last column: the current token), optional bias, act 1 = silu, residual != 0: the input is added to the
  *   result; d_state [slots][taps - 1][channels] holds a request's last inputs and is advanced by the step (by the convolution
- *   kernel itself for requests that bring one row, by a second launch for the others).
+ *   kernel itself for requests that bring one row, by a second launch for the others).  d_in_bias (optional): added to every
+ *   input row per channel (inputs before a request's start stay zero).
  *   Output in the compute type (d_out) and / or fp32 (d_out_f32).
  * vb_cast_rows: d_out [T][n] (dense, compute type) = d_in[t][0 .. n) (fp32 rows of stride ld_in).
  * vb_qk_norm_append: tail of a (q | k | v) projection: q and k RMS-normed over their whole width nq / nk with per-coordinate
@@ -710,7 +748,12 @@ int vb_pair_hash_rows(int32_t* d_rows, int32_t* d_prev_tok, const int32_t* d_ids
 int vb_short_conv(void* d_out, int ld_out, float* d_out_f32, int ld_f32, const float* d_in, int ld_in, const float* d_w,
                   const float* d_bias, float* d_state, const int32_t* d_qo_indptr, const int32_t* d_row_req, const int32_t* d_pos,
                   const int32_t* d_slots, int T, int B, int channels, int taps, int act, int residual, int out_dtype,
-                  void* stream);
+                  const float* d_in_bias, void* stream);
+/* A block's tail over up to three branches: x[t] += sum_k scale_k * (w_k ? y_k[t] / sqrt(mean(y_k[t]^2) + eps) * w_k : y_k[t])
+ * in place (fp32; y_k NULL: no such branch), d_out (optional) = x[t] / sqrt(mean(x[t]^2) + eps) * d_wn in the compute type. */
+int vb_branch_residual_norm_f32(float* d_x, const float* d_y0, const float* d_w0, float scale0, const float* d_y1,
+                                const float* d_w1, float scale1, const float* d_y2, const float* d_w2, float scale2, void* d_out,
+                                const float* d_wn, int T, int width, float eps, int out_dtype, void* stream);
 /* Hyper-connections (hyper.cu): a residual stream of `streams` copies d_xs [T][streams][width] (fp32, in place).
  *   x_t <- sum_s d_mix[s][t] x_s + d_out_c[t] (d_y + d_bias) (d_x0 given: every copy starts as that row instead; keep_streams
  *   == 0: the new copies are not written back), u = sum_s d_in_c[s] x_s (NULL: coefficients of one), then

@@ -134,10 +134,10 @@ SIGNATURES = {
     "vb_qkv_rotary_append": (c_int, [P, c_int, c_int, c_int, c_int, P, c_int, P, P, P, P, P, P, P, c_int, c_int, c_int,
                                      c_int, c_int, c_int, c_int, P, P, c_int, P]),
     "vb_window_attn": (c_int, [P, P, P, P, P, c_int, P, P, P, P, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_float,
-                               c_int, P, C.c_longlong, P, c_int, c_int, c_int, c_int, c_int, c_int, P, P]),
+                               c_int, P, C.c_longlong, P, c_int, c_int, c_int, c_int, c_int, c_int, P, c_int, c_int, P]),
     "vb_window_attn_tile_rows": (c_int, []),
     "vb_window_attn_tiled": (c_int, [P, P, P, P, P, c_int, P, P, P, P, P, P, c_int, c_int, c_int, c_int, c_int, c_int,
-                                     c_int, c_int, c_float, c_int, c_int, c_int, c_int, c_int, c_int, P, P]),
+                                     c_int, c_int, c_float, c_int, c_int, c_int, c_int, c_int, c_int, P, c_int, c_int, P]),
     "vb_decay_attn": (c_int, [P, P, P, c_int, c_int, c_int, c_int, P, P, P, P, c_int, c_int, c_int, c_int, c_int, c_int,
                               P]),
     "vb_decay_attn_tile_rows": (c_int, [c_int, c_int]),
@@ -161,7 +161,18 @@ SIGNATURES = {
     "vb_pair_hash_rows": (c_int, [P, P, P, P, P, P, P, c_int, c_int, C.c_longlong, C.c_longlong, P]),
     "vb_hyper_mix_norm": (c_int, [P, c_int, P, P, P, P, P, P, P, P, P, c_int, c_int, c_float, P, c_int, P, P, P, c_int, c_int, P]),
     "vb_short_conv": (c_int, [P, c_int, P, c_int, P, c_int, P, P, P, P, P, P, P, c_int, c_int, c_int, c_int, c_int, c_int, c_int,
-                              P]),
+                              P, P]),
+    "vb_rglru": (c_int, [P, c_int, P, P, P, P, c_int, P, P, P, c_float, P, c_int, P, P, P, P, P, P, P, c_int, c_int, c_int, c_int,
+                         c_int, c_int, c_int, c_int, c_int, P]),
+    "vb_ssd": (c_int, [P, P, P, c_int, P, c_int, P, P, P, P, c_int, P, P, P, c_int, c_int, c_int, c_int, c_int, c_int, c_int,
+                       c_int, P]),
+    "vb_ssd_tile_rows": (c_int, [c_int, c_int]),
+    "vb_ssd_scratch_floats": (C.c_longlong, [c_int, c_int, c_int, c_int]),
+    "vb_ssd_tiled": (c_int, [P, P, P, P, c_int, P, c_int, P, P, P, P, c_int, P, P, P, P, P, c_int, c_int, c_int, c_int, c_int,
+                             c_int, c_int, P]),
+    "vb_group_rmsnorm": (c_int, [P, P, P, c_int, c_int, c_int, c_float, c_int, P]),
+    "vb_moe_route_table": (c_int, [P, P, P, P, P, P, P, c_int, c_int, c_int, c_int, c_int, c_int, P]),
+    "vb_branch_residual_norm_f32": (c_int, [P, P, P, c_float, P, P, c_float, P, P, c_float, P, P, c_int, c_int, c_float, c_int, P]),
     "vb_cast_rows": (c_int, [P, P, c_int, c_int, c_int, c_int, P]),
     "vb_qk_norm_append": (c_int, [P, c_int, c_int, c_int, c_int, P, P, c_float, P, P, P, P, P, P, P, c_int, c_int, c_int, c_int,
                                   c_int, c_int, P]),
@@ -237,7 +248,8 @@ LAUNCHES = {"vb_set_pdl": 0, "vb_set_trace": 0, "vb_weight_tiles_bytes": 0, "vb_
             "vb_tensor_map_2d_bf16": 0, "vb_device_info": 0, "vb_sample": 1, "vb_update_repetition_cache": 1,
             "vb_set_gemm_smem_kb": 0, "vb_window_attn_tile_rows": 0, "vb_decay_attn_tile_rows": 0, "vb_decay_attn_tiled": 3, "vb_window_attn": 2, "vb_mingru_tiled": 3, "vb_mingru_scratch_floats": 0,
             "vb_short_conv": 2, "vb_selective_scan_tiled": 3, "vb_selective_scan_piece_rows": 0,
-            "vb_selective_scan_scratch_floats": 0, "vb_sigmoid_attn": 1}
+            "vb_selective_scan_scratch_floats": 0, "vb_sigmoid_attn": 1, "vb_ssd_tiled": 3, "vb_ssd_tile_rows": 0,
+            "vb_ssd_scratch_floats": 0}
 launch_counter = [0]
 
 

@@ -22,7 +22,7 @@ INCLUDE = os.path.join(os.path.dirname(HERE), "include")
 
 SOURCES = ["api.cu", "elementwise.cu", "attn.cu", "prefill_attn.cu", "prefill_attn_tc.cu", "kvcopy.cu", "encoder.cu", "gemm.cu", "sampler.cu", "snac.cu", "snac_mma.cu",
            "multicodebook.cu", "mimi.cu", "codec.cu", "norm_linear.cu", "window_attn.cu", "linear_attn.cu", "gated_recurrence.cu", "moe.cu", "short_conv.cu", "sigmoid_attn.cu", "selective_scan.cu",
-           "hyper.cu"]
+           "hyper.cu", "ssd.cu"]
 # subsets of the sources that serve one family of models: a first run that only needs that family compiles only these
 # (into lib/libvoxb200_<profile>.so; entry points of the other sources are absent from it)
 _TEXT = ["api.cu", "elementwise.cu", "gemm.cu", "sampler.cu", "norm_linear.cu", "window_attn.cu"]
@@ -31,7 +31,9 @@ PROFILES = {"text": _TEXT + ["linear_attn.cu", "moe.cu"],           # attention 
             # attention + short convolutions + pooled-window sigmoid attention + selective scan + mixtures of experts
             "text_conv": _TEXT + ["moe.cu", "short_conv.cu", "sigmoid_attn.cu", "selective_scan.cu"],
             # attention + short convolutions + hyper-connected streams, dense feed-forward
-            "text_hyper": _TEXT + ["short_conv.cu", "hyper.cu"]}
+            "text_hyper": _TEXT + ["short_conv.cu", "hyper.cu"],
+            # attention + short convolutions + gated linear recurrence + state-space duality + mixtures of experts
+            "text_ssd": _TEXT + ["moe.cu", "short_conv.cu", "gated_recurrence.cu", "ssd.cu"]}
 NVCC_FLAGS = [
     "-gencode", "arch=compute_100a,code=sm_100a", "-O3", "-lineinfo", "-std=c++17",
     "-Xcompiler", "-fPIC",

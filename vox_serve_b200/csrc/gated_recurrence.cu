@@ -1,5 +1,6 @@
-// Element-wise gated recurrences over a per-request fp32 state slot (minGRU: gates that read only the current token).
+// Element-wise gated recurrences over a per-request fp32 state slot, whose gates read only the current token.
 //
+// minGRU:
 //   z_t = sigmoid(pz_t + bz)                       update gate
 //   c_t = u + 1/2 (u >= 0), sigmoid(u) (u < 0)     candidate, u = px_t + bx   (positive and continuous at 0)
 //   S_t = (1 - z_t) S_(t-1) + z_t c_t              per channel, S = 0 before a request's position 0
@@ -13,6 +14,15 @@
 //   vb_mingru_tiled  prompt portions cut into pieces of rows: the recurrence S_t = a_t S_(t-1) + b_t composes as
 //                    (A, B) = (prod a, local end state from zero), so pieces are summarised in parallel, a short scan over a
 //                    request's pieces carries the state in, and the pieces then produce their rows in parallel.
+//
+// Real-gated linear recurrent unit (Griffin: De et al., "Griffin: Mixing Gated Linear Recurrences with Local Attention for
+// Efficient Language Models"):
+//   r_t = sigmoid(R_b u_t + br),  i_t = sigmoid(I_b u_t + bi)     in every block b of neighbouring channels, R_b, I_b square
+//   log a_t = -c r_t softplus(lam),  S_t = a_t S_(t-1) + sqrt(1 - a_t^2) i_t u_t,  out_t = S_t * gelu_tanh(y_t + by)
+//   vb_rglru         one kernel forms the gates of all rows (block-diagonal products: tensor cores for bf16 matrices whose
+//                    blocks are multiples of 16 channels, with u split into two bf16 terms so that a product keeps 16 bits of
+//                    u's mantissa; fp32 FMAs otherwise) and finishes the rows of requests that bring one row; the others leave
+//                    (a, sqrt(1 - a^2) i u) per channel, which a walk in order or the piecewise scan above turns into rows.
 #include "../../include/vb_api.h"
 #define VB_PDL_FAMILY 1
 #include "common.cuh"
@@ -181,6 +191,188 @@ __global__ void __launch_bounds__(128) mingru_tile_out_kernel(MinGruParams p) {
   }
 }
 
+// ------------------------------------------------------------------------------------------------------------------
+// real-gated linear recurrent unit
+// ------------------------------------------------------------------------------------------------------------------
+struct RgLruParams {
+  const float* u;         // [T][ld_u]: the recurrence's input
+  int ld_u;
+  const void* w;          // [blocks][2 * bs][bs]: the matrix of r, then that of i
+  const float* bias;      // [blocks][2 * bs]
+  const float* lam;       // [C]
+  const float* y;         // [T][ld_y]: the other branch before its bias and gelu
+  int ld_y;
+  const float* y_bias;    // [C] or nullptr
+  float* state;           // [slots][C]
+  void* out;              // [T][ld_out]
+  int ld_out;
+  float* ab;              // [T][2][C]: a, then the scaled input, of the rows that this kernel does not finish
+  const int32_t* qo_indptr;
+  const int32_t* row_req;
+  const int32_t* pos;
+  const int32_t* slots;
+  int T, B, C, bs;
+  float c;
+  int n_tiles, tile_rows; // piecewise form
+  const int32_t* tile_req;
+  const int32_t* tile_row0;
+  const float* scratch;   // [pieces][2][C]: carry-ins after the scan
+};
+
+__device__ __forceinline__ float gelu_tanh_f(float v) {
+  return 0.5f * v * (1.f + tanhf(0.79788456080286536f * (v + 0.044715f * v * v * v)));
+}
+__device__ __forceinline__ float softplus_f(float v) { return fmaxf(v, 0.f) + log1pf(expf(-fabsf(v))); }
+
+template <typename CT>
+__device__ __forceinline__ void rg_out(const RgLruParams& p, int t, int ch, float S) {
+  const float y = p.y[static_cast<size_t>(t) * p.ld_y + ch] + (p.y_bias ? p.y_bias[ch] : 0.f);
+  mg_store<CT>(p.out, static_cast<size_t>(t) * p.ld_out + ch, S * gelu_tanh_f(y));
+}
+
+// gate pre-activations zr, zi of (row, channel) -> the decay and scaled input; a request's only row is finished here
+template <typename CT>
+__device__ __forceinline__ void rg_finish(const RgLruParams& p, int t, int ch, float zr, float zi) {
+  const float la = -p.c * mg_sigmoid(zr) * softplus_f(p.lam[ch]);
+  const float a = expf(la);
+  const float v = sqrtf(-expm1f(2.f * la)) * mg_sigmoid(zi) * p.u[static_cast<size_t>(t) * p.ld_u + ch];
+  const int b = p.row_req[t];
+  if (p.qo_indptr[b + 1] - p.qo_indptr[b] == 1) {
+    float* st = p.state + static_cast<size_t>(p.slots[b]) * p.C + ch;
+    const float S = fmaf(a, p.pos[t] == 0 ? 0.f : *st, v);
+    *st = S;
+    rg_out<CT>(p, t, ch, S);
+  } else {
+    float* o = p.ab + static_cast<size_t>(t) * 2 * p.C + ch;
+    o[0] = a;
+    o[p.C] = v;
+  }
+}
+
+// any block size, fp32 FMAs in k order: CTA = 32 rows x 32 channels of one block (both gates)
+constexpr int RG_R = 32, RG_CH = 32, RG_K = 32;
+
+template <typename WT, typename CT>
+__global__ void __launch_bounds__(256) rglru_gates_kernel(RgLruParams p) {
+  __shared__ float Us[RG_R][RG_K + 1];
+  __shared__ float Ws[2][RG_CH][RG_K + 1];
+  pdl_sync();
+  const int per = (p.bs + RG_CH - 1) / RG_CH, blk = blockIdx.x / per, c0 = (blockIdx.x - blk * per) * RG_CH;
+  const int t0 = blockIdx.y * RG_R, tid = threadIdx.x, tx = tid & 31, ty = tid >> 5;
+  const WT* W = static_cast<const WT*>(p.w) + static_cast<size_t>(blk) * 2 * p.bs * p.bs;
+  float acc[2][4];
+#pragma unroll
+  for (int i = 0; i < 4; ++i) acc[0][i] = acc[1][i] = 0.f;
+  for (int k0 = 0; k0 < p.bs; k0 += RG_K) {
+    const int k = k0 + tx;
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+      const int r = ty + 8 * i;
+      Us[r][tx] = (t0 + r < p.T && k < p.bs) ? p.u[static_cast<size_t>(t0 + r) * p.ld_u + blk * p.bs + k] : 0.f;
+#pragma unroll
+      for (int g = 0; g < 2; ++g) {
+        float w = 0.f;
+        if (c0 + r < p.bs && k < p.bs) {
+          const WT v = W[static_cast<size_t>(g * p.bs + c0 + r) * p.bs + k];
+          if constexpr (sizeof(WT) == 4) w = v;
+          else w = __bfloat162float(v);
+        }
+        Ws[g][r][tx] = w;
+      }
+    }
+    __syncthreads();
+#pragma unroll 8
+    for (int kk = 0; kk < RG_K; ++kk) {
+      const float wr = Ws[0][tx][kk], wi = Ws[1][tx][kk];
+#pragma unroll
+      for (int i = 0; i < 4; ++i) {
+        const float u = Us[ty + 8 * i][kk];
+        acc[0][i] = fmaf(u, wr, acc[0][i]);
+        acc[1][i] = fmaf(u, wi, acc[1][i]);
+      }
+    }
+    __syncthreads();
+  }
+  if (c0 + tx >= p.bs) return;
+  const float* bias = p.bias + static_cast<size_t>(blk) * 2 * p.bs + c0 + tx;
+#pragma unroll
+  for (int i = 0; i < 4; ++i) {
+    const int t = t0 + ty + 8 * i;
+    if (t < p.T) rg_finish<CT>(p, t, blk * p.bs + c0 + tx, acc[0][i] + bias[0], acc[1][i] + bias[p.bs]);
+  }
+}
+
+// requests that bring several rows, in order: one thread per (request, channel)
+template <typename CT>
+__global__ void __launch_bounds__(128) rglru_walk_kernel(RgLruParams p) {
+  pdl_sync();
+  const int ch = blockIdx.x * 128 + threadIdx.x, b = blockIdx.y;
+  if (ch >= p.C) return;
+  const int r0 = p.qo_indptr[b], r1 = p.qo_indptr[b + 1];
+  if (r1 - r0 < 2) return;
+  float* st = p.state + static_cast<size_t>(p.slots[b]) * p.C + ch;
+  float S = p.pos[r0] == 0 ? 0.f : *st;
+  for (int t = r0; t < r1; ++t) {
+    const float* ab = p.ab + static_cast<size_t>(t) * 2 * p.C + ch;
+    S = fmaf(ab[0], S, ab[p.C]);
+    rg_out<CT>(p, t, ch, S);
+  }
+  *st = S;
+}
+
+// the pieces' summaries (product of the decays, end state from zero); vb::mingru_tile_scan_kernel turns them into carry-ins
+__global__ void __launch_bounds__(128) rglru_piece_sum_kernel(RgLruParams p, float* __restrict__ scratch) {
+  pdl_sync();
+  const int ch = blockIdx.x * 128 + threadIdx.x, ppt = p.tile_rows / MG_ROWS;
+  const int tile = blockIdx.y / ppt, piece = blockIdx.y - tile * ppt;
+  if (ch >= p.C) return;
+  const int r0 = p.tile_row0[tile] + piece * MG_ROWS;
+  const int n = min(min(r0 + MG_ROWS, p.tile_row0[tile] + p.tile_rows), p.qo_indptr[p.tile_req[tile] + 1]) - r0;
+  float* s = scratch + static_cast<size_t>(blockIdx.y) * 2 * p.C;
+  if (n <= 0) { s[ch] = 1.f; s[p.C + ch] = 0.f; return; }
+  float a[MG_ROWS], v[MG_ROWS];
+#pragma unroll
+  for (int i = 0; i < MG_ROWS; ++i) {
+    const float* ab = p.ab + static_cast<size_t>(r0 + min(i, n - 1)) * 2 * p.C + ch;
+    a[i] = ab[0];
+    v[i] = ab[p.C];
+  }
+  float A = 1.f, S = 0.f;
+#pragma unroll
+  for (int i = 0; i < MG_ROWS; ++i)
+    if (i < n) { A *= a[i]; S = fmaf(a[i], S, v[i]); }
+  s[ch] = A;
+  s[p.C + ch] = S;
+}
+
+template <typename CT>
+__global__ void __launch_bounds__(128) rglru_piece_out_kernel(RgLruParams p) {
+  pdl_sync();
+  const int ch = blockIdx.x * 128 + threadIdx.x, ppt = p.tile_rows / MG_ROWS;
+  const int tile = blockIdx.y / ppt, piece = blockIdx.y - tile * ppt;
+  if (ch >= p.C) return;
+  const int r0 = p.tile_row0[tile] + piece * MG_ROWS;
+  const int n = min(min(r0 + MG_ROWS, p.tile_row0[tile] + p.tile_rows), p.qo_indptr[p.tile_req[tile] + 1]) - r0;
+  if (n <= 0) return;
+  float a[MG_ROWS], v[MG_ROWS], y[MG_ROWS];
+#pragma unroll
+  for (int i = 0; i < MG_ROWS; ++i) {
+    const int t = r0 + min(i, n - 1);
+    const float* ab = p.ab + static_cast<size_t>(t) * 2 * p.C + ch;
+    a[i] = ab[0];
+    v[i] = ab[p.C];
+    y[i] = p.y[static_cast<size_t>(t) * p.ld_y + ch];
+  }
+  const float yb = p.y_bias ? p.y_bias[ch] : 0.f;
+  float S = p.scratch[static_cast<size_t>(blockIdx.y) * 2 * p.C + ch];
+#pragma unroll
+  for (int i = 0; i < MG_ROWS; ++i)
+    if (i < n) {
+      S = fmaf(a[i], S, v[i]);
+      mg_store<CT>(p.out, static_cast<size_t>(r0 + i) * p.ld_out + ch, S * gelu_tanh_f(y[i] + yb));
+    }
+}
+
 }  // namespace vb
 
 using namespace vb;
@@ -216,6 +408,48 @@ int vb_mingru_tiled(void* d_out, float* d_state, float* d_scratch, const float* 
   VB_LAUNCH_PDL(mingru_tile_scan_kernel, dim3(cx, B), 128, 0, stream, p);
   if (out_dtype == 1) VB_LAUNCH_PDL(mingru_tile_out_kernel<float>, dim3(cx, pieces), 128, 0, stream, p);
   else VB_LAUNCH_PDL(mingru_tile_out_kernel<bf16>, dim3(cx, pieces), 128, 0, stream, p);
+  return 0;
+}
+
+int vb_rglru(void* d_out, int ld_out, float* d_state, float* d_ab, float* d_scratch, const float* d_u, int ld_u, const void* d_w,
+             const float* d_bias, const float* d_lam, float c, const float* d_y, int ld_y, const float* d_y_bias,
+             const int32_t* d_qo_indptr, const int32_t* d_row_req, const int32_t* d_pos, const int32_t* d_slots,
+             const int32_t* d_tile_req, const int32_t* d_tile_row0, int n_tiles, int tile_rows, int T, int B, int width,
+             int blocks, int multi_rows, int w_dtype, int out_dtype, void* stream) {
+  VB_CHECK_ARG(d_out && d_state && d_u && d_w && d_bias && d_lam && d_y && d_qo_indptr && d_row_req && d_pos && d_slots &&
+               (!multi_rows || d_ab), "vb_rglru: null pointer");
+  VB_CHECK_ARG(width > 0 && blocks > 0 && width % blocks == 0 && ld_u >= width && ld_y >= width && ld_out >= width,
+               "vb_rglru: width %d in %d blocks", width, blocks);
+  VB_CHECK_ARG(n_tiles <= 0 || (d_tile_req && d_tile_row0 && d_scratch && tile_rows > 0 && tile_rows % MG_ROWS == 0),
+               "vb_rglru: the piecewise form needs tiles of a multiple of %d rows and scratch", MG_ROWS);
+  if (T <= 0 || B <= 0) return 0;
+  const int bs = width / blocks;
+  RgLruParams p{d_u, ld_u, d_w, d_bias, d_lam, d_y, ld_y, d_y_bias, d_state, d_out, ld_out, d_ab, d_qo_indptr, d_row_req, d_pos,
+                d_slots, T, B, width, bs, c, n_tiles, tile_rows, d_tile_req, d_tile_row0, d_scratch};
+  const bool f32 = out_dtype == 1;
+  const dim3 grid(blocks * ((bs + RG_CH - 1) / RG_CH), (T + RG_R - 1) / RG_R);
+  if (w_dtype == 1) {
+    if (f32) VB_LAUNCH_PDL((rglru_gates_kernel<float, float>), grid, 256, 0, stream, p);
+    else VB_LAUNCH_PDL((rglru_gates_kernel<float, bf16>), grid, 256, 0, stream, p);
+  } else {
+    if (f32) VB_LAUNCH_PDL((rglru_gates_kernel<bf16, float>), grid, 256, 0, stream, p);
+    else VB_LAUNCH_PDL((rglru_gates_kernel<bf16, bf16>), grid, 256, 0, stream, p);
+  }
+  if (!multi_rows) return 0;
+  const int cx = (width + 127) / 128;
+  if (n_tiles <= 0) {
+    if (f32) VB_LAUNCH_PDL(rglru_walk_kernel<float>, dim3(cx, B), 128, 0, stream, p);
+    else VB_LAUNCH_PDL(rglru_walk_kernel<bf16>, dim3(cx, B), 128, 0, stream, p);
+    return 0;
+  }
+  const int pieces = n_tiles * (tile_rows / MG_ROWS);
+  MinGruParams sp{};
+  sp.state = d_state; sp.qo_indptr = d_qo_indptr; sp.pos = d_pos; sp.slots = d_slots; sp.B = B; sp.width = width;
+  sp.tile_req = d_tile_req; sp.tile_row0 = d_tile_row0; sp.n_tiles = n_tiles; sp.tile_rows = tile_rows; sp.scratch = d_scratch;
+  VB_LAUNCH_PDL(rglru_piece_sum_kernel, dim3(cx, pieces), 128, 0, stream, p, d_scratch);
+  VB_LAUNCH_PDL(mingru_tile_scan_kernel, dim3(cx, B), 128, 0, stream, sp);
+  if (f32) VB_LAUNCH_PDL(rglru_piece_out_kernel<float>, dim3(cx, pieces), 128, 0, stream, p);
+  else VB_LAUNCH_PDL(rglru_piece_out_kernel<bf16>, dim3(cx, pieces), 128, 0, stream, p);
   return 0;
 }
 

@@ -7,6 +7,8 @@
 //                   ranks by the sum of its two largest corrected scores; experts outside count as -inf), and WEIGHTED
 //                   by their uncorrected s divided by the chosen experts' sum (+ 1e-20).  Also the shared expert's
 //                   per-token gate sigmoid(w_sg . h) when asked
+//   vb_moe_route_table  no scores: the token's id picks its experts from a table [vocab][top], each weighs 1 / top; also the
+//                   shared expert's per-token gate sigmoid(w_sg . h) when asked
 //   vb_moe_group    counting sort (shared-memory counters, one CTA) of the (token, choice) pairs by expert: row_off[E + 1], the token of every sorted row and
 //                   the sorted row of every (token, choice)
 //   vb_moe_scale_dense  the dense form for tensor-core projections: every expert runs on every token as ONE stacked
@@ -201,6 +203,49 @@ __global__ void __launch_bounds__(256) moe_route_sigmoid_kernel(int32_t* __restr
   if (lane < top) wts[t * top + lane] = normalize ? my_val / (denom + 1e-20f) : my_val;
 }
 
+// one warp per token
+template <typename XT>
+__global__ void __launch_bounds__(128) moe_route_table_kernel(int32_t* __restrict__ idx, float* __restrict__ wts,
+                                                              float* __restrict__ shared_gate, const int32_t* __restrict__ ids,
+                                                              const int32_t* __restrict__ table, const XT* __restrict__ h,
+                                                              const float* __restrict__ wsg, int T, int W, int vocab, int E,
+                                                              int top) {
+  pdl_sync();
+  const int t = blockIdx.x * 4 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
+  if (t >= T) return;
+  const int32_t* row = table + static_cast<size_t>(min(max(ids[t], 0), vocab - 1)) * top;
+  for (int c = lane; c < top; c += 32) {
+    idx[static_cast<size_t>(t) * top + c] = min(max(row[c], 0), E - 1);
+    wts[static_cast<size_t>(t) * top + c] = 1.f / top;
+  }
+  if (wsg == nullptr) return;
+  const XT* x = h + static_cast<size_t>(t) * W;
+  float s = 0.f;
+  if ((W & 7) == 0) {
+    for (int i = lane * 8; i < W; i += 256) {
+      const float4 a = *reinterpret_cast<const float4*>(wsg + i), b = *reinterpret_cast<const float4*>(wsg + i + 4);
+      float v[8];
+      if constexpr (sizeof(XT) == 4) {
+        const float4 p = *reinterpret_cast<const float4*>(x + i), q = *reinterpret_cast<const float4*>(x + i + 4);
+        v[0] = p.x; v[1] = p.y; v[2] = p.z; v[3] = p.w; v[4] = q.x; v[5] = q.y; v[6] = q.z; v[7] = q.w;
+      } else {
+        const uint4 p = *reinterpret_cast<const uint4*>(x + i);
+        v[0] = bf16_lo(p.x); v[1] = bf16_hi(p.x); v[2] = bf16_lo(p.y); v[3] = bf16_hi(p.y);
+        v[4] = bf16_lo(p.z); v[5] = bf16_hi(p.z); v[6] = bf16_lo(p.w); v[7] = bf16_hi(p.w);
+      }
+      s = fmaf(v[0], a.x, s); s = fmaf(v[1], a.y, s); s = fmaf(v[2], a.z, s); s = fmaf(v[3], a.w, s);
+      s = fmaf(v[4], b.x, s); s = fmaf(v[5], b.y, s); s = fmaf(v[6], b.z, s); s = fmaf(v[7], b.w, s);
+    }
+  } else {
+    for (int i = lane; i < W; i += 32) {
+      if constexpr (sizeof(XT) == 4) s = fmaf(x[i], wsg[i], s);
+      else s = fmaf(__bfloat162float(x[i]), wsg[i], s);
+    }
+  }
+  s = warp_sum(s);
+  if (lane == 0) shared_gate[t] = 1.f / (1.f + expf(-s));
+}
+
 // single CTA: E <= 1024 experts, any number of pairs
 __global__ void __launch_bounds__(1024) moe_group_kernel(int32_t* __restrict__ row_off, int32_t* __restrict__ sorted_token,
                                                          int32_t* __restrict__ pair_row, const int32_t* __restrict__ idx,
@@ -366,6 +411,19 @@ int vb_moe_route_groups(int32_t* d_idx, float* d_wts, float* d_shared_gate, cons
   VB_CHECK_ARG(smem <= 48 * 1024, "vb_moe_route_sigmoid: width %d too large", width);
   if (h_dtype == 1) VB_LAUNCH_PDL(moe_route_sigmoid_kernel<float>, T, 256, smem, stream, d_idx, d_wts, d_shared_gate, static_cast<const float*>(d_h), d_router_w, d_correction, d_shared_gate_w, width, experts, top, ng, keep, softmax_scores, rank_by_max, normalize);
   else VB_LAUNCH_PDL(moe_route_sigmoid_kernel<__nv_bfloat16>, T, 256, smem, stream, d_idx, d_wts, d_shared_gate, static_cast<const __nv_bfloat16*>(d_h), d_router_w, d_correction, d_shared_gate_w, width, experts, top, ng, keep, softmax_scores, rank_by_max, normalize);
+  return 0;
+}
+
+int vb_moe_route_table(int32_t* d_idx, float* d_wts, float* d_shared_gate, const int32_t* d_ids, const int32_t* d_table,
+                       const void* d_h, const float* d_shared_gate_w, int T, int width, int vocab, int experts, int top,
+                       int h_dtype, void* stream) {
+  VB_CHECK_ARG(d_idx && d_wts && d_ids && d_table && vocab > 0 && (!d_shared_gate_w || (d_shared_gate && d_h && width > 0)),
+               "vb_moe_route_table: bad arguments");
+  VB_CHECK_ARG(experts >= 1 && experts <= 1024 && top >= 1 && top <= 32 && top <= experts,
+               "vb_moe_route_table: experts %d (<= 1024), top %d (<= 32, <= experts)", experts, top);
+  if (T <= 0) return 0;
+  if (h_dtype == 1) VB_LAUNCH_PDL(moe_route_table_kernel<float>, (T + 3) / 4, 128, 0, stream, d_idx, d_wts, d_shared_gate, d_ids, d_table, static_cast<const float*>(d_h), d_shared_gate_w, T, width, vocab, experts, top);
+  else VB_LAUNCH_PDL(moe_route_table_kernel<__nv_bfloat16>, (T + 3) / 4, 128, 0, stream, d_idx, d_wts, d_shared_gate, d_ids, d_table, static_cast<const __nv_bfloat16*>(d_h), d_shared_gate_w, T, width, vocab, experts, top);
   return 0;
 }
 

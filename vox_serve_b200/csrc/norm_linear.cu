@@ -219,6 +219,110 @@ __global__ void __launch_bounds__(256) gated_residual_norm_kernel(float* __restr
   }
 }
 
+// The tail of a block that adds up to three branches to the stream at once, some of them normed first, in place on the fp32 row:
+//   x[t] += sum_k scale_k * (w_k ? y_k[t] / sqrt(mean(y_k[t]^2) + eps) * w_k : y_k[t])
+//   out[t] = x[t] / sqrt(mean(x[t]^2) + eps) * w      (optional: what the next block reads)
+struct BranchTailParams {
+  float* x;
+  const float* y[3];          // nullptr: no such branch
+  const float* w[3];          // nullptr: the branch enters as it is
+  float scale[3];
+  void* out;
+  const float* wn;
+  int W;
+  float eps;
+};
+
+// NV > 0: rows that move in 16-byte pieces, at most NV pieces per thread, kept in registers between the passes; NV == 0: any row
+template <typename OT, int NV>
+__global__ void __launch_bounds__(256) branch_residual_norm_kernel(BranchTailParams p) {
+  __shared__ float red[64];
+  int phase = 0;
+  pdl_sync();
+  const size_t o = static_cast<size_t>(blockIdx.x) * p.W;
+  if constexpr (NV > 0) {
+    const int n4 = p.W >> 2;
+    float4 x[NV], y[3][NV];
+    float q[3] = {0.f, 0.f, 0.f};
+#pragma unroll
+    for (int k = 0; k < 3; ++k)
+      if (p.y[k])
+#pragma unroll
+        for (int i = 0; i < NV; ++i) {
+          const int c = threadIdx.x + 256 * i;
+          y[k][i] = c < n4 ? *reinterpret_cast<const float4*>(p.y[k] + o + 4 * c) : make_float4(0.f, 0.f, 0.f, 0.f);
+        }
+#pragma unroll
+    for (int i = 0; i < NV; ++i) {
+      const int c = threadIdx.x + 256 * i;
+      x[i] = c < n4 ? *reinterpret_cast<const float4*>(p.x + o + 4 * c) : make_float4(0.f, 0.f, 0.f, 0.f);
+    }
+#pragma unroll
+    for (int k = 0; k < 3; ++k) {
+      if (p.y[k] == nullptr) continue;
+      float rs = p.scale[k];
+      if (p.w[k]) {
+#pragma unroll
+        for (int i = 0; i < NV; ++i) {
+          q[k] = fmaf(y[k][i].x, y[k][i].x, q[k]); q[k] = fmaf(y[k][i].y, y[k][i].y, q[k]);
+          q[k] = fmaf(y[k][i].z, y[k][i].z, q[k]); q[k] = fmaf(y[k][i].w, y[k][i].w, q[k]);
+        }
+        rs /= sqrtf(block_sum(q[k], red, phase) / p.W + p.eps);
+      }
+#pragma unroll
+      for (int i = 0; i < NV; ++i) {
+        const int c = threadIdx.x + 256 * i;
+        float4 w = make_float4(rs, rs, rs, rs);
+        if (p.w[k] && c < n4) {
+          const float4 v = *reinterpret_cast<const float4*>(p.w[k] + 4 * c);
+          w.x *= v.x; w.y *= v.y; w.z *= v.z; w.w *= v.w;
+        }
+        x[i].x = fmaf(w.x, y[k][i].x, x[i].x); x[i].y = fmaf(w.y, y[k][i].y, x[i].y);
+        x[i].z = fmaf(w.z, y[k][i].z, x[i].z); x[i].w = fmaf(w.w, y[k][i].w, x[i].w);
+      }
+    }
+    float s = 0.f;
+#pragma unroll
+    for (int i = 0; i < NV; ++i) {
+      const int c = threadIdx.x + 256 * i;
+      if (c < n4) *reinterpret_cast<float4*>(p.x + o + 4 * c) = x[i];
+      s = fmaf(x[i].x, x[i].x, s); s = fmaf(x[i].y, x[i].y, s); s = fmaf(x[i].z, x[i].z, s); s = fmaf(x[i].w, x[i].w, s);
+    }
+    if (p.out == nullptr) return;
+    const float rs = 1.f / sqrtf(block_sum(s, red, phase) / p.W + p.eps);
+#pragma unroll
+    for (int i = 0; i < NV; ++i) {
+      const int c = threadIdx.x + 256 * i;
+      if (c < n4) {
+        const float4 w = *reinterpret_cast<const float4*>(p.wn + 4 * c);
+        store4<OT>(static_cast<OT*>(p.out) + o + 4 * c, x[i].x * rs * w.x, x[i].y * rs * w.y, x[i].z * rs * w.z, x[i].w * rs * w.w);
+      }
+    }
+  } else {
+    extern __shared__ float row[];
+    float rs[3];
+    for (int k = 0; k < 3; ++k) {
+      rs[k] = p.scale[k];
+      if (p.y[k] == nullptr || p.w[k] == nullptr) continue;
+      float q = 0.f;
+      for (int i = threadIdx.x; i < p.W; i += 256) q = fmaf(p.y[k][o + i], p.y[k][o + i], q);
+      rs[k] /= sqrtf(block_sum(q, red, phase) / p.W + p.eps);
+    }
+    float s = 0.f;
+    for (int i = threadIdx.x; i < p.W; i += 256) {
+      float v = p.x[o + i];
+      for (int k = 0; k < 3; ++k)
+        if (p.y[k]) v = fmaf(rs[k] * (p.w[k] ? p.w[k][i] : 1.f), p.y[k][o + i], v);
+      p.x[o + i] = v;
+      row[i] = v;
+      s = fmaf(v, v, s);
+    }
+    if (p.out == nullptr) return;
+    const float r = 1.f / sqrtf(block_sum(s, red, phase) / p.W + p.eps);
+    for (int i = threadIdx.x; i < p.W; i += 256) static_cast<OT*>(p.out)[o + i] = from_f<OT>(row[i] * r * p.wn[i]);
+  }
+}
+
 // ROWS rows per CTA: the side matrices are read once per CTA and serve all of its rows (long steps).  A row's result
 // depends on nothing but the row; between the one-row form (16 warps) and the four-row form (8 warps) only the order in
 // which the norms' sums of squares are added differs.
@@ -833,6 +937,40 @@ int vb_rms_postnorm_residual_f32(float* d_x, const float* d_y, const float* d_w,
   } else {
     if (smem > 48 * 1024) VB_CHECK_CUDA(cudaFuncSetAttribute(rms_postnorm_residual_kernel<bf16>, cudaFuncAttributeMaxDynamicSharedMemorySize, VB_MAX_DYN_SMEM));
     VB_LAUNCH_PDL(rms_postnorm_residual_kernel<bf16>, T, 256, smem, stream, d_x, d_y, d_w, static_cast<bf16*>(d_out), width, eps);
+  }
+  return 0;
+}
+
+int vb_branch_residual_norm_f32(float* d_x, const float* d_y0, const float* d_w0, float scale0, const float* d_y1,
+                                const float* d_w1, float scale1, const float* d_y2, const float* d_w2, float scale2, void* d_out,
+                                const float* d_wn, int T, int width, float eps, int out_dtype, void* stream) {
+  VB_CHECK_ARG(d_x && width > 0 && (!d_out || d_wn), "vb_branch_residual_norm_f32: bad arguments");
+  if (T <= 0) return 0;
+  BranchTailParams p{d_x, {d_y0, d_y1, d_y2}, {d_w0, d_w1, d_w2}, {scale0, scale1, scale2}, d_out, d_wn, width, eps};
+  auto al16 = [](const void* q) { return q == nullptr || reinterpret_cast<uintptr_t>(q) % 16 == 0; };
+  const bool vec = width % 4 == 0 && al16(d_x) && al16(d_y0) && al16(d_y1) && al16(d_y2) && al16(d_w0) && al16(d_w1) && al16(d_w2) &&
+                   al16(d_wn) && (!d_out || reinterpret_cast<uintptr_t>(d_out) % 8 == 0);
+  const int pieces = vec ? (width / 4 + 255) / 256 : 0;
+  const bool f32 = out_dtype == 1;
+  if (pieces == 1) {
+    if (f32) VB_LAUNCH_PDL((branch_residual_norm_kernel<float, 1>), T, 256, 0, stream, p);
+    else VB_LAUNCH_PDL((branch_residual_norm_kernel<bf16, 1>), T, 256, 0, stream, p);
+  } else if (pieces == 2) {
+    if (f32) VB_LAUNCH_PDL((branch_residual_norm_kernel<float, 2>), T, 256, 0, stream, p);
+    else VB_LAUNCH_PDL((branch_residual_norm_kernel<bf16, 2>), T, 256, 0, stream, p);
+  } else if (pieces == 3 || pieces == 4) {
+    if (f32) VB_LAUNCH_PDL((branch_residual_norm_kernel<float, 4>), T, 256, 0, stream, p);
+    else VB_LAUNCH_PDL((branch_residual_norm_kernel<bf16, 4>), T, 256, 0, stream, p);
+  } else {
+    const size_t smem = static_cast<size_t>(width) * sizeof(float);
+    VB_CHECK_ARG(smem <= static_cast<size_t>(VB_MAX_DYN_SMEM) - 1024, "vb_branch_residual_norm_f32: width %d too large", width);
+    if (f32) {
+      if (smem > 40 * 1024) VB_CHECK_CUDA(cudaFuncSetAttribute(branch_residual_norm_kernel<float, 0>, cudaFuncAttributeMaxDynamicSharedMemorySize, VB_MAX_DYN_SMEM - 1024));
+      VB_LAUNCH_PDL((branch_residual_norm_kernel<float, 0>), T, 256, smem, stream, p);
+    } else {
+      if (smem > 40 * 1024) VB_CHECK_CUDA(cudaFuncSetAttribute(branch_residual_norm_kernel<bf16, 0>, cudaFuncAttributeMaxDynamicSharedMemorySize, VB_MAX_DYN_SMEM - 1024));
+      VB_LAUNCH_PDL((branch_residual_norm_kernel<bf16, 0>), T, 256, smem, stream, p);
+    }
   }
   return 0;
 }

@@ -4,7 +4,8 @@
 //                                                                       request's position 0 are zero)
 //   out_t  = act(y_t) (+ u_t: the residual form h + conv(h))
 //
-// u is a column range of fp32 rows (the residual stream, or the rows of a fused projection), so several convolutions over
+// u is a column range of fp32 rows (the residual stream, or the rows of a fused projection; a bias per channel -- the
+// projection's -- may be added to it first, inputs before a request's start stay zero), so several convolutions over
 // neighbouring columns of one projection run as ONE call with their weights stacked.  A request's last taps - 1 inputs live
 // in an fp32 slot [taps - 1][C]; rows whose taps reach before the step's first row read them from there.  A request that
 // brings one row has its slot shifted by that row's own thread; the slots of the others are rewritten by a second kernel after
@@ -30,6 +31,7 @@ struct ShortConvParams {
   int ld_in;
   const float* w;         // [C][taps]
   const float* bias;      // [C] or nullptr
+  const float* in_bias;   // [C] added to every input row, or nullptr
   float* state;           // [slots][taps - 1][C]
   void* out;              // [T][ld_out] compute type, or nullptr
   int ld_out;
@@ -57,15 +59,16 @@ __global__ void __launch_bounds__(256) short_conv_kernel(ShortConvParams p) {
   const int b = p.row_req[t], r = t - p.qo_indptr[b], ps = p.pos[t], K = p.taps - 1;
   const float* st = p.state + (static_cast<size_t>(p.slots[b]) * K) * p.C + c;
   const float* w = p.w + static_cast<size_t>(c) * p.taps;
+  const float ib = p.in_bias ? p.in_bias[c] : 0.f;
   float acc = p.bias ? p.bias[c] : 0.f;
   for (int j = 0; j < p.taps; ++j) {
     const int back = K - j;
     if (ps - back < 0) continue;
-    const float u = r - back >= 0 ? p.in[static_cast<size_t>(t - back) * p.ld_in + c] : st[static_cast<size_t>(r + j) * p.C];
+    const float u = r - back >= 0 ? p.in[static_cast<size_t>(t - back) * p.ld_in + c] + ib : st[static_cast<size_t>(r + j) * p.C];
     acc = fmaf(w[j], u, acc);
   }
   if (p.act == 1) acc = acc / (1.f + expf(-acc));
-  const float cur = p.in[static_cast<size_t>(t) * p.ld_in + c];
+  const float cur = p.in[static_cast<size_t>(t) * p.ld_in + c] + ib;
   if (p.residual) acc += cur;
   if (p.out) sc_store<CT>(p.out, static_cast<size_t>(t) * p.ld_out + c, acc);
   if (p.out_f32) p.out_f32[static_cast<size_t>(t) * p.ld_f32 + c] = acc;
@@ -98,10 +101,11 @@ __global__ void __launch_bounds__(256) short_conv_rows_kernel(ShortConvParams p)
   if (c >= p.C) return;
   constexpr int K = TAPS - 1;
   float u[SC_RPT + K], w[TAPS];
+  const float ib = p.in_bias ? p.in_bias[c] : 0.f;
 #pragma unroll
   for (int i = 0; i < SC_RPT + K; ++i) {
     const int t = t0 - K + i;
-    u[i] = (t >= 0 && t < p.T) ? p.in[static_cast<size_t>(t) * p.ld_in + c] : 0.f;
+    u[i] = (t >= 0 && t < p.T) ? p.in[static_cast<size_t>(t) * p.ld_in + c] + ib : 0.f;
   }
 #pragma unroll
   for (int j = 0; j < TAPS; ++j) w[j] = p.w[static_cast<size_t>(c) * TAPS + j];
@@ -144,12 +148,13 @@ __global__ void __launch_bounds__(SC_VTHREADS) short_conv_rows4_kernel(ShortConv
   constexpr int K = TAPS - 1;
   const int c = (blockIdx.x * SC_VTHREADS + threadIdx.x) * 4, t0 = blockIdx.y * SC_VRPT;
   if (c >= p.C) { pdl_sync(); return; }
-  float w[4][TAPS], bias[4];
+  float w[4][TAPS], bias[4], ib[4];
 #pragma unroll
   for (int e = 0; e < 4; ++e) {
 #pragma unroll
     for (int j = 0; j < TAPS; ++j) w[e][j] = p.w[static_cast<size_t>(c + e) * TAPS + j];
     bias[e] = p.bias ? p.bias[c + e] : 0.f;
+    ib[e] = p.in_bias ? p.in_bias[c + e] : 0.f;
   }
   pdl_sync();
   float u[SC_VRPT + K][4];
@@ -158,7 +163,7 @@ __global__ void __launch_bounds__(SC_VTHREADS) short_conv_rows4_kernel(ShortConv
     const int t = t0 - K + i;
     float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
     if (t >= 0 && t < p.T) v = *reinterpret_cast<const float4*>(p.in + static_cast<size_t>(t) * p.ld_in + c);
-    u[i][0] = v.x; u[i][1] = v.y; u[i][2] = v.z; u[i][3] = v.w;
+    u[i][0] = v.x + ib[0]; u[i][1] = v.y + ib[1]; u[i][2] = v.z + ib[2]; u[i][3] = v.w + ib[3];
   }
   const int b0 = p.row_req[t0];
   const bool inside = t0 - p.qo_indptr[b0] >= K && p.row_req[min(t0 + SC_VRPT, p.T) - 1] == b0;
@@ -210,6 +215,7 @@ __global__ void __launch_bounds__(256) short_conv_state_kernel(ShortConvParams p
   if (n <= 0 || K <= 0) return;
   if (n == 1 && p.single_inline) return;        // (shifted by the row's own thread)
   const int p0 = p.pos[r0];
+  const float ib = p.in_bias ? p.in_bias[c] : 0.f;
   float* st = p.state + (static_cast<size_t>(p.slots[b]) * K) * p.C + c;
   float keep[SC_MAX_TAPS];
 #pragma unroll
@@ -217,7 +223,7 @@ __global__ void __launch_bounds__(256) short_conv_state_kernel(ShortConvParams p
     if (i >= K) break;
     const int src = n + i;                      // index into [old slot (K) | rows (n)]
     float v = 0.f;
-    if (p0 - K + src >= 0) v = src < K ? st[static_cast<size_t>(src) * p.C] : p.in[static_cast<size_t>(r0 + src - K) * p.ld_in + c];
+    if (p0 - K + src >= 0) v = src < K ? st[static_cast<size_t>(src) * p.C] : p.in[static_cast<size_t>(r0 + src - K) * p.ld_in + c] + ib;
     keep[i] = v;
   }
 #pragma unroll
@@ -284,14 +290,14 @@ int vb_pair_hash_rows(int32_t* d_rows, int32_t* d_prev_tok, const int32_t* d_ids
 int vb_short_conv(void* d_out, int ld_out, float* d_out_f32, int ld_f32, const float* d_in, int ld_in, const float* d_w,
                   const float* d_bias, float* d_state, const int32_t* d_qo_indptr, const int32_t* d_row_req, const int32_t* d_pos,
                   const int32_t* d_slots, int T, int B, int channels, int taps, int act, int residual, int out_dtype,
-                  void* stream) {
+                  const float* d_in_bias, void* stream) {
   VB_CHECK_ARG(d_in && d_w && d_state && d_qo_indptr && d_row_req && d_pos && d_slots && (d_out || d_out_f32),
                "vb_short_conv: null pointer");
   VB_CHECK_ARG(channels > 0 && taps >= 1 && taps <= SC_MAX_TAPS && (act == 0 || act == 1) && ld_in >= channels,
                "vb_short_conv: channels %d, taps %d (1..%d), act %d", channels, taps, SC_MAX_TAPS, act);
   if (T <= 0 || B <= 0) return 0;
   const bool rows_form = T >= 64 && taps >= 2 && taps <= 4;
-  ShortConvParams p{d_in, ld_in, d_w, d_bias, d_state, d_out, ld_out, d_out_f32, ld_f32, d_qo_indptr, d_row_req, d_pos, d_slots,
+  ShortConvParams p{d_in, ld_in, d_w, d_bias, d_in_bias, d_state, d_out, ld_out, d_out_f32, ld_f32, d_qo_indptr, d_row_req, d_pos, d_slots,
                     T, B, channels, taps, act, residual, rows_form ? 0 : 1};
   const int cx = (channels + 255) / 256;
   const dim3 rows_grid(cx, (T + SC_RPT - 1) / SC_RPT);

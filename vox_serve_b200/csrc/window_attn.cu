@@ -18,7 +18,8 @@
 //                        query head, a shared rotated key part behind a latent, and the combination of two score maps per head.
 // Besides the sliding window the kernels take a chunk mask (a position sees the keys of its own block of positions), per-token
 // strides of the two caches (a value that is a leading slice of the key row), key heads that share a value head, an fp32
-// output beside bf16 operands, and a sink per head: one more term e^sink in the softmax's denominator, a key without a value.
+// output beside bf16 operands, a sink per head: one more term e^sink in the softmax's denominator, a key without a value,
+// the first tokens of a sequence kept visible to every later position (keep_first), and a gate per head instead of per value.
 // Cache layout per layer: K [pages][page_size][kv_heads][dim], V [pages][page_size][kv_heads][vdim] unless strides say otherwise.
 #include "../../include/vb_api.h"
 #define VB_PDL_FAMILY 1
@@ -387,7 +388,30 @@ struct WindowAttnParams {
   int splits;                 // grouped kernel: key tiles are dealt round-robin to `splits` CTAs per (row, key/value head)
   float* part;                // [T][H][splits][vdim + 2]: unnormalised output, running max, running sum of every split
   const float* sink;          // [H] score of a further key without a value that enters every row's denominator, or nullptr
+  int keep;                   // positions 0 .. keep - 1 are visible to every later position, however far (0: none)
+  int head_gate;              // the gate holds one value per head (column h) instead of one per output value
 };
+
+// a gate's value for output value d of head h of a row (column h, or h * vdim + d)
+__device__ __forceinline__ float wa_gate(const WindowAttnParams& p, const float* __restrict__ row, int h, int d) {
+  return 1.f / (1.f + expf(-row[p.head_gate ? h : h * p.vdim + d]));
+}
+
+// The keys that the rows of a tile walk: [0, min(keep, lo)) in n0 steps of KT keys, then [lo, last] -- where lo is the first
+// key that the tile's first row sees otherwise.  Without kept tokens (or where they touch lo) there is one range.
+struct WaRange {
+  int lo, pre, n0, n;         // pre = min(keep, lo): keys of the first range; n0 its steps; n all steps
+  __device__ __forceinline__ int first(int i, int kt) const { return i < n0 ? i * kt : lo + (i - n0) * kt; }
+  __device__ __forceinline__ int end(int i, int last) const { return i < n0 ? pre : last + 1; }      // keys at or past it are not of this range
+};
+__device__ __forceinline__ WaRange wa_range(const WindowAttnParams& p, int lo, int last, int kt) {
+  WaRange r;
+  r.lo = lo;
+  r.pre = min(p.keep, lo);
+  r.n0 = (r.pre + kt - 1) / kt;
+  r.n = r.n0 + (last - lo + kt) / kt;
+  return r;
+}
 
 // what a row's accumulated values are multiplied by, from its running maximum and sum: 1 / l, or with a sink
 // e^(m - M) / (l e^(m - M) + e^(sink - M)), M = max(m, sink)
@@ -507,9 +531,11 @@ __global__ void __launch_bounds__(WA_WARPS * 32) window_attn_kernel(WindowAttnPa
   float m = -INFINITY, l = 0.f, acc[WA_MAXU];
 #pragma unroll
   for (int u = 0; u < WA_MAXU; ++u) acc[u] = 0.f;
-  for (int c = lo; c <= ps; c += 32) {
+  const WaRange rg = wa_range(p, lo, ps, 32);
+  for (int it = 0; it < rg.n; ++it) {
+    const int c = rg.first(it, 32), c_end = rg.end(it, ps);
     const int kj = c + lane;
-    const bool ok = kj <= ps;
+    const bool ok = kj < c_end;
     int tok = 0;
     float s = -INFINITY;
     if (ok) {
@@ -523,7 +549,7 @@ __global__ void __launch_bounds__(WA_WARPS * 32) window_attn_kernel(WindowAttnPa
     m = m_new;
 #pragma unroll
     for (int u = 0; u < WA_MAXU; ++u) acc[u] *= corr;
-    const int n = min(32, ps - c + 1);
+    const int n = min(32, c_end - c);
     for (int jj = 0; jj < n; ++jj) {
       const float pv = __shfl_sync(0xffffffffu, pj, jj);
       const int tk = __shfl_sync(0xffffffffu, tok, jj);
@@ -537,13 +563,13 @@ __global__ void __launch_bounds__(WA_WARPS * 32) window_attn_kernel(WindowAttnPa
   }
   const float inv = wa_inv(p, h, m, l);
   const size_t out0 = static_cast<size_t>(t) * p.H * p.vdim + h * p.vdim;
-  const float* gate = p.gate ? p.gate + static_cast<size_t>(t) * p.ld_gate + h * p.vdim : nullptr;
+  const float* gate = p.gate ? p.gate + static_cast<size_t>(t) * p.ld_gate : nullptr;
 #pragma unroll
   for (int u = 0; u < WA_MAXU; ++u) {
     const int d = lane + 32 * u;
     if (d < p.vdim) {
       float o = acc[u] * inv;
-      if (gate) o *= 1.f / (1.f + expf(-gate[d]));
+      if (gate) o *= wa_gate(p, gate, h, d);
       wa_store<CT>(p, out0 + d, o);
     }
   }
@@ -590,9 +616,10 @@ __global__ void __launch_bounds__(256) window_attn_tiled_kernel(WindowAttnParams
 #pragma unroll
   for (int u = 0; u < WT_MAXD; ++u) acc[u] = 0.f;
   const int nd = (dv + 3) / 4;
-  for (int c0 = lo; c0 <= pos_last; c0 += WT_KEYS) {
+  const WaRange rg = wa_range(p, lo, pos_last, WT_KEYS);
+  for (int it = 0; it < rg.n; ++it) {
     __syncthreads();
-    const int valid = min(WT_KEYS, pos_last - c0 + 1);
+    const int c0 = rg.first(it, WT_KEYS), valid = min(WT_KEYS, rg.end(it, pos_last) - c0);
     load_rows_f32<CT>(Ks, dkp, kc, pages, p.page_size, p.k_ld, g * dk, dk, c0, WT_KEYS, valid, tid, 256);
     load_rows_f32<CT>(Vs, dvp, vc, pages, p.page_size, p.v_ld, gv * dv, dv, c0, WT_KEYS, valid, tid, 256);
     __syncthreads();
@@ -606,7 +633,7 @@ __global__ void __launch_bounds__(256) window_attn_tiled_kernel(WindowAttnParams
       const float* qr = Qs + r * dkp;
       const float* kr = Ks + kk * dkp;
       for (int d = 0; d < dk; ++d) a = fmaf(qr[d], kr[d], a);
-      const bool vis = row_ok && kj <= my_pos && kj >= my_lo;
+      const bool vis = row_ok && kk < valid && kj <= my_pos && (kj >= my_lo || kj < p.keep);
       s[e] = vis ? a : -INFINITY;
       mx = fmaxf(mx, s[e]);
     }
@@ -644,13 +671,13 @@ __global__ void __launch_bounds__(256) window_attn_tiled_kernel(WindowAttnParams
   const int t = row0 + r;
   const float inv = wa_inv(p, h, m, l);
   const size_t out0 = static_cast<size_t>(t) * p.H * dv + h * dv;
-  const float* gate = p.gate ? p.gate + static_cast<size_t>(t) * p.ld_gate + h * dv : nullptr;
+  const float* gate = p.gate ? p.gate + static_cast<size_t>(t) * p.ld_gate : nullptr;
 #pragma unroll
   for (int u = 0; u < WT_MAXD; ++u) {
     const int d = c + 4 * u;
     if (u < nd && d < dv) {
       float o = acc[u] * inv;
-      if (gate) o *= 1.f / (1.f + expf(-gate[d]));
+      if (gate) o *= wa_gate(p, gate, h, d);
       wa_store<CT>(p, out0 + d, o);
     }
   }
@@ -693,9 +720,10 @@ __global__ void __launch_bounds__(128) window_attn_group_kernel(WindowAttnParams
     for (int v = 0; v < WD_VU; ++v) acc[u][v] = 0.f;
   }
   const int S = p.splits, sidx = blockIdx.z;
-  for (int c0 = lo + sidx * WD_KEYS; c0 <= ps; c0 += S * WD_KEYS) {
+  const WaRange rg = wa_range(p, lo, ps, WD_KEYS);
+  for (int it = sidx; it < rg.n; it += S) {
     __syncthreads();
-    const int nk = min(WD_KEYS, ps - c0 + 1);
+    const int c0 = rg.first(it, WD_KEYS), nk = min(WD_KEYS, rg.end(it, ps) - c0);
     load_rows_f32<CT>(Ks, dkp, kc, pages, p.page_size, p.k_ld, g * dk, dk, c0, WD_KEYS, nk, tid, 128);
     load_rows_f32<CT>(Vs, dvp, vc, pages, p.page_size, p.v_ld, gv * dv, dv, c0, WD_KEYS, nk, tid, 128);
     __syncthreads();
@@ -750,13 +778,13 @@ __global__ void __launch_bounds__(128) window_attn_group_kernel(WindowAttnParams
     }
     const float inv = wa_inv(p, h, m[u], l[u]);
     const size_t out0 = static_cast<size_t>(t) * p.H * dv + h * dv;
-    const float* gate = p.gate ? p.gate + static_cast<size_t>(t) * p.ld_gate + h * dv : nullptr;
+    const float* gate = p.gate ? p.gate + static_cast<size_t>(t) * p.ld_gate : nullptr;
 #pragma unroll
     for (int v = 0; v < WD_VU; ++v) {
       const int d = lane + 32 * v;
       if (d < dv) {
         float o = acc[u][v] * inv;
-        if (gate) o *= 1.f / (1.f + expf(-gate[d]));
+        if (gate) o *= wa_gate(p, gate, h, d);
         wa_store<CT>(p, out0 + d, o);
       }
     }
@@ -782,11 +810,11 @@ __global__ void __launch_bounds__(64) window_attn_merge_kernel(WindowAttnParams 
   }
   __syncthreads();
   const size_t out0 = static_cast<size_t>(t) * p.H * dv + h * dv;
-  const float* gate = p.gate ? p.gate + static_cast<size_t>(t) * p.ld_gate + h * dv : nullptr;
+  const float* gate = p.gate ? p.gate + static_cast<size_t>(t) * p.ld_gate : nullptr;
   for (int d = threadIdx.x; d < dv; d += blockDim.x) {
     float o = 0.f;
     for (int s = 0; s < S; ++s) o = fmaf(pt[s * (dv + 2) + d], wgt[s], o);
-    if (gate) o *= 1.f / (1.f + expf(-gate[d]));
+    if (gate) o *= wa_gate(p, gate, h, d);
     wa_store<CT>(p, out0 + d, o);
   }
 }
@@ -859,14 +887,14 @@ __global__ void __launch_bounds__(128) window_attn_mma_kernel(WindowAttnParams p
   const int stage_elems = FN * (ldk + dv + 8);
   // thread t copies 16-byte piece (t % 16) + 16 n of rows (t / 16) + 8 m: the page lookup and the row's cache offset are
   // computed once per row and serve its K and its V pieces
-  auto issue_tile = [&](int c0, int stage) {
+  auto issue_tile = [&](int c0, int c_end, int stage) {
     __nv_bfloat16* Kd = Ks + stage * stage_elems;
     __nv_bfloat16* Vd = Kd + FN * ldk;
     const int piece = tid & 15;
 #pragma unroll 2
     for (int kk = tid >> 4; kk < FN; kk += 8) {
       const int kj = c0 + kk;
-      const bool ok = kj <= pos_last;
+      const bool ok = kj < c_end;
       const int kq = ok ? kj : pos_last;                 // (a valid address also for the zero-filled rows)
       const int pg = kq / p.page_size;
       const size_t tok = static_cast<size_t>(pages[pg]) * p.page_size + (kq - pg * p.page_size);
@@ -882,12 +910,13 @@ __global__ void __launch_bounds__(128) window_attn_mma_kernel(WindowAttnParams p
     asm volatile("cp.async.commit_group;" ::: "memory");
   };
   __syncthreads();                    // every warp holds its Q fragments: the first stage may be overwritten
-  const int c_first = lo + sidx * FN, c_step = FN * S;
-  if (c_first <= pos_last) issue_tile(c_first, 0);
+  const WaRange rg = wa_range(p, lo, pos_last, FN);
+  if (sidx < rg.n) issue_tile(rg.first(sidx, FN), rg.end(sidx, pos_last), 0);
   int stage = 0;
-  for (int c0 = c_first; c0 <= pos_last; c0 += c_step, stage ^= 1) {
-    if (c0 + c_step <= pos_last) {
-      issue_tile(c0 + c_step, stage ^ 1);
+  for (int it = sidx; it < rg.n; it += S, stage ^= 1) {
+    const int c0 = rg.first(it, FN), c_end = rg.end(it, pos_last);
+    if (it + S < rg.n) {
+      issue_tile(rg.first(it + S, FN), rg.end(it + S, pos_last), stage ^ 1);
       asm volatile("cp.async.wait_group 1;" ::: "memory");
     } else {
       asm volatile("cp.async.wait_group 0;" ::: "memory");
@@ -898,7 +927,7 @@ __global__ void __launch_bounds__(128) window_attn_mma_kernel(WindowAttnParams p
     // a warp whose 16 rows see nothing of this tile has no work in it
     const int w_first = pos0 + warp * 16 * pstep, w_last = min(pos0 + (warp * 16 + 15) * pstep, pos_last);
     const int w_lo = wa_first_key(p, w_first);
-    const bool idle = warp * 16 >= nrows || c0 > w_last || c0 + FN - 1 < w_lo;
+    const bool idle = warp * 16 >= nrows || c0 > w_last || (c0 + FN - 1 < w_lo && c0 >= p.keep);
     if (!idle) {
     float sc[FN / 8][4];
 #pragma unroll
@@ -921,7 +950,8 @@ __global__ void __launch_bounds__(128) window_attn_mma_kernel(WindowAttnParams p
 #pragma unroll
       for (int e = 0; e < 4; ++e) {
         const int kj = c0 + n * 8 + (lane & 3) * 2 + (e & 1);
-        const bool vis = e < 2 ? (okA && kj <= posA && kj >= loA) : (okB && kj <= posB && kj >= loB);
+        const bool vis = kj < c_end && (e < 2 ? (okA && kj <= posA && (kj >= loA || kj < p.keep))
+                                              : (okB && kj <= posB && (kj >= loB || kj < p.keep)));
         const float v = vis ? sc[n][e] * p.scale : -INFINITY;
         sc[n][e] = v;
         if (e < 2) mxA = fmaxf(mxA, v);
@@ -1008,10 +1038,10 @@ __global__ void __launch_bounds__(128) window_attn_mma_kernel(WindowAttnParams p
         const int t = row0 + (half ? rB : rA);          // (row_heads: token * H + head)
         float x0 = o[n][2 * half] * (half ? iB : iA), x1 = o[n][2 * half + 1] * (half ? iB : iA);
         if (p.gate) {
-          const float* gt = p.row_heads ? p.gate + static_cast<size_t>(t / p.H) * p.ld_gate + (t % p.H) * dv + d
-                                        : p.gate + static_cast<size_t>(t) * p.ld_gate + h * dv + d;
-          x0 *= 1.f / (1.f + expf(-gt[0]));
-          x1 *= 1.f / (1.f + expf(-gt[1]));
+          const float* gt = p.gate + static_cast<size_t>(p.row_heads ? t / p.H : t) * p.ld_gate;
+          const int hg = p.row_heads ? t % p.H : h;
+          x0 *= wa_gate(p, gt, hg, d);
+          x1 *= wa_gate(p, gt, hg, d + 1);
         }
         const size_t oi = static_cast<size_t>(t) * HH * dv + h * dv + d;
         if (p.out_f32) *reinterpret_cast<float2*>(static_cast<float*>(p.out) + oi) = make_float2(x0, x1);
@@ -1153,7 +1183,8 @@ int vb_window_attn(void* d_out, const void* d_q, const void* d_k_cache, const vo
                    int ld_gate, const int32_t* d_row_req, const int32_t* d_pos, const int32_t* d_page_indptr,
                    const int32_t* d_page_indices, int T, int H, int G, int dim, int vdim, int page_size, int window,
                    float scale, int dtype, float* d_part, long long part_floats, const int32_t* d_row_list, int head_rows,
-                   int chunk, int k_ld, int v_ld, int v_share, int out_f32, const float* d_sink, void* stream) {
+                   int chunk, int k_ld, int v_ld, int v_share, int out_f32, const float* d_sink, int keep_first,
+                   int head_gate, void* stream) {
   VB_CHECK_ARG(d_out && d_q && d_k_cache && d_v_cache && d_row_req && d_pos && d_page_indptr && d_page_indices,
                "vb_window_attn: null pointer");
   VB_CHECK_ARG(H > 0 && G > 0 && H % G == 0 && dim > 0 && vdim > 0 && vdim <= 32 * WA_MAXU && page_size > 0,
@@ -1165,7 +1196,7 @@ int vb_window_attn(void* d_out, const void* d_q, const void* d_k_cache, const vo
   if (v_ld <= 0) v_ld = (G / v_share) * vdim;
   WindowAttnParams p{d_q, d_k_cache, d_v_cache, d_out, d_gate, ld_gate, d_row_req, d_pos, d_page_indptr, d_page_indices,
                      nullptr, nullptr, nullptr, T, H, G, dim, vdim, page_size, window, chunk, k_ld, v_ld, v_share, out_f32,
-                     scale, d_row_list, 0, 1, d_part, d_sink};
+                     scale, d_row_list, 0, 1, d_part, d_sink, max(keep_first, 0), head_gate};
   const int R = H / G;
   const bool mma_ok = dtype == 0 && dim % 16 == 0 && vdim % 16 == 0 && dim <= 16 * F_KB && vdim <= 8 * F_NT &&
                       k_ld % 8 == 0 && v_ld % 8 == 0;
@@ -1229,7 +1260,8 @@ int vb_window_attn_tiled(void* d_out, const void* d_q, const void* d_k_cache, co
                          int ld_gate, const int32_t* d_pos, const int32_t* d_page_indptr, const int32_t* d_page_indices,
                          const int32_t* d_qo_indptr, const int32_t* d_tile_req, const int32_t* d_tile_row0, int n_tiles,
                          int T, int H, int G, int dim, int vdim, int page_size, int window, float scale, int dtype,
-                         int chunk, int k_ld, int v_ld, int v_share, int out_f32, const float* d_sink, void* stream) {
+                         int chunk, int k_ld, int v_ld, int v_share, int out_f32, const float* d_sink, int keep_first,
+                   int head_gate, void* stream) {
   VB_CHECK_ARG(d_out && d_q && d_k_cache && d_v_cache && d_pos && d_page_indptr && d_page_indices && d_qo_indptr &&
                d_tile_req && d_tile_row0, "vb_window_attn_tiled: null pointer");
   VB_CHECK_ARG(H > 0 && G > 0 && H % G == 0 && dim > 0 && vdim > 0 && vdim <= 4 * WT_MAXD && page_size > 0,
@@ -1241,7 +1273,7 @@ int vb_window_attn_tiled(void* d_out, const void* d_q, const void* d_k_cache, co
   if (v_ld <= 0) v_ld = (G / v_share) * vdim;
   WindowAttnParams p{d_q, d_k_cache, d_v_cache, d_out, d_gate, ld_gate, nullptr, d_pos, d_page_indptr, d_page_indices,
                      d_qo_indptr, d_tile_req, d_tile_row0, T, H, G, dim, vdim, page_size, window, chunk, k_ld, v_ld, v_share,
-                     out_f32, scale, nullptr, 0, 1, nullptr, d_sink};
+                     out_f32, scale, nullptr, 0, 1, nullptr, d_sink, max(keep_first, 0), head_gate};
   dim3 grid(n_tiles, H);
   if (dtype == 0 && dim % 16 == 0 && vdim % 16 == 0 && dim <= 16 * F_KB && vdim <= 8 * F_NT && k_ld % 8 == 0 && v_ld % 8 == 0) {
     const size_t msmem = 2 * static_cast<size_t>(FN) * (dim + 8 + vdim + 8) * sizeof(__nv_bfloat16);      // two stages

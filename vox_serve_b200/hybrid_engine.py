@@ -28,7 +28,10 @@ token-pair embedding and a tied head (``_forward_post``).  A fifth, ``hyper`` (h
 copies; a sublayer reads a weighted sum of them through a norm and an input convolution with state, and its output enters all of
 them beside a mix of the old ones), carries latent attention with a query latent and a rotated part, and grouped-head attention
 with projection biases, values of unit RMS, a factor per head on the scores and a sink in the softmax's denominator
-(``_forward_hyper`` at the end of this file).
+(``_forward_hyper``).  Parallel blocks may share ONE norm between their sublayers (``shared_norm``,
+``_forward_shared_norm`` at the end of this file); such stacks carry window attention with projection biases and a gate per head,
+state-space duality (Mamba-2), and a pair of mixers whose outputs are normed before they are added -- window attention that keeps
+the first tokens visible and has a learned sink, beside a real-gated linear recurrent unit -- with experts looked up by token id.
 
 Precision: ``dtype`` bfloat16 keeps projections' operands, q / k / v, the page cache and the attention output in bf16 with
 fp32 accumulation; norms, softmax, router, residual, recurrent state, decays and the lightning path after its projection
@@ -117,10 +120,14 @@ class WindowAttentionConfig:
     rotary: Optional[RotaryConfig] = None
     v_mix: bool = False
     gate: bool = True
-    bias: bool = False                    # biases on the q, k, v and output projections
+    bias: bool = False                    # biases on the q, k, v and (o_bias) output projections
+    o_bias: bool = True
     value_norm: bool = False              # every value head divided by its root mean square over vdim (cached so)
     head_factor: bool = False             # scores times one number per query head
     sink: Optional[float] = None          # score of a further key without a value in every softmax (0: one joins the denominator)
+    learned_sink: bool = False            # ... one stored number per head instead
+    keep_first: int = 0                   # the first so many positions stay visible to every later one, outside the window too
+    head_gate: bool = False               # (with gate) one sigmoid gate per head instead of one per output value
 
 
 @dataclass
@@ -193,6 +200,48 @@ class MixerPairConfig:
 
 
 @dataclass
+class GatedLinearRecurrenceConfig:
+    """Real-gated linear recurrent unit behind a short convolution, times a gelu branch: y = gelu_tanh(W_y h + b), u =
+    conv(W_x h + b); r, i = sigmoid of u through block-diagonal matrices (``blocks`` equal parts of the channels);
+    log a = -c r softplus(lam), S_t = a S_(t-1) + sqrt(1 - a^2) i u over an fp32 state of ``width`` values per request; output
+    W_o (S * y)."""
+    width: int
+    blocks: int
+    conv: int
+    c: float = 8.0
+
+
+@dataclass
+class StateSpaceConfig:
+    """State-space duality (Mamba-2): [z | x | B | C | dt] = W_in h; x, B, C through a causal convolution (bias) and silu;
+    dt = softplus(dt + bias); per head S_t = exp(-exp(A_log) dt) S_(t-1) + dt B_t x_t^T over an fp32 state [state, vdim],
+    y = S^T C + D x, B and C shared by the heads of a group; y * silu(z), RMS-normed in ``norm_groups`` equal parts, then W_o."""
+    heads: int
+    vdim: int
+    state: int
+    groups: int
+    conv: int
+    norm_groups: int = 1
+
+    @property
+    def inner(self) -> int:
+        return self.heads * self.vdim
+
+    @property
+    def conv_channels(self) -> int:
+        return self.inner + 2 * self.groups * self.state
+
+
+@dataclass
+class NormedPairConfig:
+    """Two mixers side by side on the same input, each through its own output projection and RMS norm over the model's width; the
+    result is scale * (left + right)."""
+    left: WindowAttentionConfig
+    right: GatedLinearRecurrenceConfig
+    scale: float = 0.5
+
+
+@dataclass
 class PairEmbedConfig:
     """A second embedding of (previous token, token) pairs: row (prev * mul_prev + token * mul_cur) mod buckets of a table of
     buckets + 1 rows, whose last row serves a sequence's first token."""
@@ -252,7 +301,7 @@ class MoEConfig:
     act: str = "silu_glu"                 # "silu_glu": down(silu(gate h) * up h); "clamped_glu": down(g sigmoid(slope g) (u + 1))
     #                                       with g = min(gate h, limit), u = clamp(up h, +-limit); else down(act(up h)) as
     #                                       DenseMLPConfig.act
-    router: str = "softmax"               # "softmax": top logits, softmax over the chosen.  "sigmoid": sigmoid scores, chosen
+    router: str = "softmax"               # "table": the token's id picks its experts from a stored table, weights 1 / top.  "softmax": top logits, softmax over the chosen.  "sigmoid": sigmoid scores, chosen
     #                                       by score + correction within the kept groups, weights = chosen scores / their sum.
     #                                       "softmax_all": scores = softmax over ALL experts, the largest within the kept
     #                                       groups chosen, weights = the chosen scores as they are
@@ -265,7 +314,8 @@ class MoEConfig:
 
 @dataclass
 class HybridLayerConfig:
-    kind: str                             # "attention" | "lightning" | "latent" | "diff_attention" | "mingru" | "mixer_pair"
+    kind: str                             # "attention" | "lightning" | "latent" | "diff_attention" | "mingru" | "mixer_pair" |
+    #                                       "state_space" | "normed_pair"
     mixer: Any
     mlp: Any = None                       # MoEConfig | DenseMLPConfig | GluMLPConfig | None
 
@@ -286,6 +336,7 @@ class HybridConfig:
     norm: str = "layernorm"               # "layernorm" (weight and bias) | "rmsnorm" (weight) | "rmsnorm_scalar" (one number) |
     #                                       "rmsnorm_offset" (the stored weight is an offset from one: x / rms * (1 + w))
     residual_mult: float = 1.0            # m of the parallel form
+    shared_norm: bool = False             # parallel form: both sublayers read ONE norm of the stream (norm1)
     positions: int = 0                    # rows of the learned position table added to the embedding (0: none)
     side_dim: int = 0                     # per-token side input of every block (parallel form): dims per layer (0: none)
     logit_softcap: float = 0.0            # logits <- cap * tanh(logits / cap) (0: none)
@@ -437,6 +488,9 @@ class HybridWeights:
                 continue
             if cfg.block == "hyper":
                 self.layers.append(self._load_hyper_layer(sd, p, i, L, norm))
+                continue
+            if cfg.block == "parallel" and cfg.shared_norm:
+                self.layers.append(self._load_shared_norm_layer(sd, p, i, L, norm))
                 continue
             if cfg.block == "parallel":
                 w: Dict[str, Any] = {"norm1": vec(p + "norm1")}
@@ -620,25 +674,7 @@ class HybridWeights:
         if L.kind == "latent":
             self._load_latent(sd, p, i, m, w)
         elif L.kind == "attention":
-            nq, nk, nv = m.heads * m.dim, m.kv_heads * m.dim, m.kv_heads * m.vdim
-            w["qkvg"] = mat(*[p + "mix." + n for n in (("q", "k", "v", "g") if m.gate else ("q", "k", "v"))])
-            w["o"] = mat(p + "mix.o")
-            if (tuple(w["qkvg"].shape) != (nq + nk + nv + (m.heads * m.vdim if m.gate else 0), W) or
-                    tuple(sd[p + "mix.q"].shape) != (nq, W) or tuple(sd[p + "mix.k"].shape) != (nk, W) or
-                    tuple(w["o"].shape) != (W, m.heads * m.vdim)):
-                raise VoxB200Error(f"layer {i}: attention shapes do not match the configuration")
-            if m.bias:
-                w["qkv_b"] = torch.cat([vec(p + f"mix.{n}.b") for n in ("q", "k", "v")], 0).contiguous()
-                w["o_b"] = vec(p + "mix.o.b")
-                if w["qkv_b"].numel() != nq + nk + nv or w["o_b"].numel() != W:
-                    raise VoxB200Error(f"layer {i}: attention bias shapes do not match the configuration")
-            if m.head_factor:
-                w["head_factor"] = vec(p + "mix.temp")
-                if w["head_factor"].numel() != m.heads:
-                    raise VoxB200Error(f"layer {i}: one score factor per head")
-            if m.sink is not None:
-                w["sink"] = torch.full((m.heads,), m.sink, dtype=F32, device=self.device)
-            w["qkvg"], w["o"] = dense(w["qkvg"]), dense(w["o"])
+            w["qkvg"], w["o"] = (dense(t) for t in self._attention_weights(sd, p + "mix.", i, m, w))
         else:
             raise VoxB200Error(f"layer {i}: mixer '{L.kind}' is not available in hyper-connected blocks")
         f = L.mlp
@@ -649,6 +685,91 @@ class HybridWeights:
                     tuple(sd[p + "mlp.down"].shape) != (W, f.ff)):
                 raise VoxB200Error(f"layer {i}: feed-forward shapes do not match the configuration")
             w["gu"], w["down"] = self._gate_up(p + "mlp.gate", p + "mlp.up"), dense(mat(p + "mlp.down"))
+        return w
+
+    def _attention_weights(self, sd, p: str, i: int, m: "WindowAttentionConfig", w: Dict[str, Any]):
+        """``<p>{q, k, v, g?, o}`` -> (q | k | v (| g) stacked, o), neither re-tiled; into w: biases ``{q,k,v}.b`` stacked like the
+        columns and ``o.b``, the factors ``temp`` [H], the sinks (a constant, or ``sink`` [H])."""
+        mat, vec, W = self._mat, self._vec, self.cfg.width
+        nq, nk, nv = m.heads * m.dim, m.kv_heads * m.dim, m.kv_heads * m.vdim
+        ng = 0 if not m.gate else (m.heads if m.head_gate else m.heads * m.vdim)
+        qkvg, o = mat(*[p + n for n in (("q", "k", "v", "g") if m.gate else ("q", "k", "v"))]), mat(p + "o")
+        if (tuple(qkvg.shape) != (nq + nk + nv + ng, W) or tuple(sd[p + "q"].shape) != (nq, W) or
+                tuple(sd[p + "k"].shape) != (nk, W) or tuple(sd[p + "v"].shape) != (nv, W) or tuple(o.shape) != (W, m.heads * m.vdim)):
+            raise VoxB200Error(f"layer {i}: attention shapes do not match the configuration")
+        if m.bias:
+            w["qkv_b"] = torch.cat([vec(p + f"{n}.b") for n in ("q", "k", "v")], 0).contiguous()
+            if m.o_bias:
+                w["o_b"] = vec(p + "o.b")
+            if w["qkv_b"].numel() != nq + nk + nv or (m.o_bias and w["o_b"].numel() != W):
+                raise VoxB200Error(f"layer {i}: attention bias shapes do not match the configuration")
+        if m.head_factor:
+            w["head_factor"] = vec(p + "temp")
+            if w["head_factor"].numel() != m.heads:
+                raise VoxB200Error(f"layer {i}: one score factor per head")
+        if m.learned_sink:
+            w["sink"] = vec(p + "sink")
+            if w["sink"].numel() != m.heads:
+                raise VoxB200Error(f"layer {i}: one sink per head")
+        elif m.sink is not None:
+            w["sink"] = torch.full((m.heads,), m.sink, dtype=F32, device=self.device)
+        return qkvg, o
+
+    def _load_shared_norm_layer(self, sd, p: str, i: int, L: "HybridLayerConfig", norm) -> Dict[str, Any]:
+        """A parallel layer whose sublayers read one norm: ``l<i>.norm1``, ``l<i>.mix.*``, ``l<i>.mlp.*``.
+          attention: q | k | v | g as ONE projection
+          state space: ``in``, ``conv[.b]``, ``dt_bias``, ``A_log``, ``D``, ``norm``, ``o``
+          normed pair: in = left.q | left.k | left.v | right.y | right.x -- ONE projection for both mixers; the recurrence's gate
+            matrices [blocks, 2 * size, size] (``ra`` above ``ri``); both output projections and norms (``left.out``, ``right.out``)
+        Feed-forward: dense (up, down) or experts without a gate matrix behind a router or a table."""
+        mat, vec, dense, cfg, W, m = self._mat, self._vec, self._dense, self.cfg, self.cfg.width, L.mixer
+        w: Dict[str, Any] = {"norm1": norm(p + "norm1")[0]}
+        x = p + "mix."
+        if L.kind == "attention":
+            w["qkvg"], w["o"] = (dense(t) for t in self._attention_weights(sd, x, i, m, w))
+        elif L.kind == "state_space":
+            C = m.conv_channels
+            win, o = mat(x + "in"), mat(x + "o")
+            w["conv"], w["conv_b"] = vec(x + "conv"), vec(x + "conv.b")
+            for n in ("dt_bias", "A_log", "D", "norm"):
+                w[n] = vec(x + n)
+            if (tuple(win.shape) != (m.inner + C + m.heads, W) or tuple(o.shape) != (W, m.inner) or tuple(w["conv"].shape) != (C, m.conv) or
+                    w["conv_b"].numel() != C or any(w[n].numel() != m.heads for n in ("dt_bias", "A_log", "D")) or
+                    w["norm"].numel() != m.inner):
+                raise VoxB200Error(f"layer {i}: state-space shapes do not match the configuration")
+            w["in"], w["o"] = dense(win), dense(o)
+        elif L.kind == "normed_pair":
+            a, r = m.left, m.right
+            if a.gate:
+                raise VoxB200Error(f"layer {i}: the attention of a normed pair has no output gate")
+            qkv, o = self._attention_weights(sd, x + "left.", i, a, w)
+            y, u, ro = mat(x + "right.y"), mat(x + "right.x"), mat(x + "right.o")
+            bs = r.width // r.blocks
+            ra, ri = mat(x + "right.ra"), mat(x + "right.ri")
+            w["conv"], w["conv_b"] = vec(x + "right.conv"), vec(x + "right.conv.b")
+            w["y_b"], w["x_b"], w["lam"] = vec(x + "right.y.b"), vec(x + "right.x.b"), vec(x + "right.lam")
+            w["left_norm"], w["right_norm"] = vec(x + "left.out"), vec(x + "right.out")
+            if (any(tuple(t.shape) != (r.width, W) for t in (y, u)) or tuple(ro.shape) != (W, r.width) or
+                    any(tuple(t.shape) != (r.blocks, bs, bs) for t in (ra, ri)) or tuple(w["conv"].shape) != (r.width, r.conv) or
+                    any(w[n].numel() != r.width for n in ("conv_b", "y_b", "x_b", "lam")) or
+                    any(w[n].numel() != W for n in ("left_norm", "right_norm"))):
+                raise VoxB200Error(f"layer {i}: gated linear recurrence shapes do not match the configuration")
+            w["in"] = dense(torch.cat([qkv, y, u], 0).contiguous())
+            w["gates"] = torch.cat([ra, ri], 1).contiguous()
+            w["gates_b"] = torch.cat([vec(x + f"right.{n}.b").reshape(r.blocks, bs) for n in ("ra", "ri")], 1).contiguous()
+            w["left_o"], w["right_o"] = dense(o), dense(ro)
+        else:
+            raise VoxB200Error(f"layer {i}: mixer '{L.kind}' is not available in blocks with one shared norm")
+        f = L.mlp
+        if isinstance(f, DenseMLPConfig):
+            up, down = mat(p + "mlp.up"), mat(p + "mlp.down")
+            if tuple(up.shape) != (f.ff, W) or tuple(down.shape) != (W, f.ff):
+                raise VoxB200Error(f"layer {i}: feed-forward shapes do not match the configuration")
+            w["up"], w["down"] = dense(up), dense(down)
+        elif isinstance(f, MoEConfig) and f.act not in ("silu_glu", "clamped_glu"):
+            self._load_plain_moe(sd, p, i, f, w)
+        elif f is not None:
+            raise VoxB200Error(f"layer {i}: blocks with one shared norm take a plain dense feed-forward or experts without a gate matrix")
         return w
 
     def _load_gated_layer(self, sd, p: str, i: int, L: "HybridLayerConfig", norm) -> Dict[str, Any]:
@@ -749,14 +870,20 @@ class HybridWeights:
         w["uv"] = uv.view(m.heads, m.vdim, m.kv_rank).contiguous()
 
     def _load_plain_moe(self, sd, p: str, i: int, f: "MoEConfig", w: Dict[str, Any]) -> None:
-        """Experts of the form down(act(up h)): ``l<i>.mlp.{router, correction, e<j>.{up, down}, shared.{up, down, sg}}``.
+        """Experts of the form down(act(up h)): ``l<i>.mlp.{router, correction, e<j>.{up, down}, shared.{up, down, sg}}``, or
+        ``table`` (int32 [vocab, top]) instead of a router.
         On tensor-core projections every expert and the shared expert are stacked into ONE up matrix (along N) and ONE down
         matrix (along K); otherwise the experts are [E, ...] stacks for the grouped linear kernel."""
         mat, vec, dense, W = self._mat, self._vec, self._dense, self.cfg.width
-        w["router"] = vec(p + "mlp.router")
-        w["correction"] = vec(p + "mlp.correction") if (p + "mlp.correction") in sd else None
-        if tuple(w["router"].shape) != (f.experts, W):
-            raise VoxB200Error(f"layer {i}: router shape does not match the configuration")
+        if f.router == "table":
+            w["table"] = sd[p + "mlp.table"].to(device=self.device, dtype=I32).contiguous()
+            if tuple(w["table"].shape) != (self.cfg.vocab, f.top) or int(w["table"].min()) < 0 or int(w["table"].max()) >= f.experts:
+                raise VoxB200Error(f"layer {i}: the expert table does not match the configuration")
+        else:
+            w["router"] = vec(p + "mlp.router")
+            w["correction"] = vec(p + "mlp.correction") if (p + "mlp.correction") in sd else None
+            if tuple(w["router"].shape) != (f.experts, W):
+                raise VoxB200Error(f"layer {i}: router shape does not match the configuration")
         if f.shared_ff and f.shared_gate:
             w["sg"] = vec(p + "mlp.shared.sg").reshape(-1)
         names = [f"e{e}" for e in range(f.experts)] + (["shared"] if f.shared_ff else [])
@@ -812,7 +939,9 @@ class HybridCache:
     per linear-attention layer a state [slots, H, dim, vdim] and per minGRU layer a state [slots, width] in fp32; per mixer
     pair K / V pages of its attention, fp32 pooled blocks [pages, ceil(page / pool), G, dim / vdim], the scan's state
     [slots, inner, N] and the last inputs of its short convolutions [slots, taps - 1, channels]; per layer of a stack with an
-    input convolution its last inputs [slots, taps - 1, width] (hyper-connected blocks: one for each sublayer); with a token-pair embedding the last token of every slot.  A layer
+    input convolution its last inputs [slots, taps - 1, width]; per state-space layer a state [slots, H, state, vdim] in fp32 and the
+    last inputs of its convolution; per normed pair K / V pages of its attention, the recurrence's state [slots, width] and the last
+    inputs of its convolution (hyper-connected blocks: one for each sublayer); with a token-pair embedding the last token of every slot.  A layer
     that a loop runs several times has one of these per pass.  Pages and slots are handed out by the worker; a slot's state is treated as zero by
     the kernels when its request starts at position 0, so nothing is cleared on reuse."""
 
@@ -844,6 +973,15 @@ class HybridCache:
                     self.k[i] = self.v[i] = self.k[m.kv_from]
             elif L.kind == "mingru":
                 self.state[i] = torch.zeros(num_slots, m.width, dtype=F32, device=device)
+            elif L.kind == "state_space":
+                self.state[i] = torch.zeros(num_slots, m.heads, m.state, m.vdim, dtype=F32, device=device)
+                self.conv[(i, "x")] = torch.zeros(num_slots, max(m.conv - 1, 1), m.conv_channels, dtype=F32, device=device)
+            elif L.kind == "normed_pair":
+                a, r = m.left, m.right
+                self.k[i] = torch.zeros(num_pages, page_size, a.kv_heads, a.dim, dtype=dtype, device=device)
+                self.v[i] = torch.zeros(num_pages, page_size, a.kv_heads, a.vdim, dtype=dtype, device=device)
+                self.state[i] = torch.zeros(num_slots, r.width, dtype=F32, device=device)
+                self.conv[(i, "x")] = torch.zeros(num_slots, max(r.conv - 1, 1), r.width, dtype=F32, device=device)
             elif L.kind == "mixer_pair":
                 a, r = m.left, m.right
                 self.k[i] = torch.zeros(num_pages, page_size, a.kv_heads, a.dim, dtype=dtype, device=device)
@@ -901,7 +1039,10 @@ class HybridEngine:
         self.w, self.cfg, self.cache, self.dtype = weights, cfg, cache, weights.dtype
         self.max_rows, self.max_out_rows = max_rows, max_out_rows
         dev, R, W, CT = weights.device, max_rows, cfg.width, weights.dtype
-        att = [L.mixer for L in cfg.layers if L.kind == "attention"]
+        npair = [L.mixer for L in cfg.layers if L.kind == "normed_pair"]
+        att = [L.mixer for L in cfg.layers if L.kind == "attention"] + [m.left for m in npair]
+        glr = [m.right for m in npair]
+        ssm = [L.mixer for L in cfg.layers if L.kind == "state_space"]
         lin = [L.mixer for L in cfg.layers if L.kind == "lightning"]
         lat = [L.mixer for L in cfg.layers if L.kind == "latent"]
         dif = [L.mixer for L in cfg.layers if L.kind == "diff_attention"]
@@ -917,7 +1058,9 @@ class HybridEngine:
         p_par = [m.left.heads * m.left.dim + m.left.kv_heads * (m.left.dim + m.left.vdim) + 2 * m.right.inner for m in par]
         p_dif = [2 * (m.heads + m.kv_heads) * m.dim + m.kv_heads * m.vdim + m.heads * m.vdim + gated for m in dif]
         p_gru = [3 * m.width + gated for m in gru]
-        hv = max([m.heads * m.vdim for m in att + lin + lat + dif] + [m.width for m in gru] +
+        p_ssm = [m.inner + m.conv_channels + m.heads for m in ssm]
+        p_pair = [m.left.heads * m.left.dim + m.left.kv_heads * (m.left.dim + m.left.vdim) + 2 * m.right.width for m in npair]
+        hv = max([m.heads * m.vdim for m in att + lin + lat + dif + ssm] + [m.width for m in gru + glr] +
                  [m.left.heads * m.left.vdim + m.right.inner for m in par] + [1])
         for m in lat:
             if m.kv_rank > 256:
@@ -928,10 +1071,21 @@ class HybridEngine:
             if m.heads % m.kv_heads or m.vdim > 256:
                 raise VoxB200Error(f"attention: {m.heads} heads on {m.kv_heads} key/value heads of {m.vdim} values "
                                    "(heads a multiple of key/value heads, at most 256 values per head)")
+        for m in att:
+            if m.heads % m.kv_heads or m.vdim > 256:
+                raise VoxB200Error(f"attention: {m.heads} heads on {m.kv_heads} key/value heads of {m.vdim} values "
+                                   "(heads a multiple of key/value heads, at most 256 values per head)")
+        for m in glr:
+            if m.blocks < 1 or m.width % m.blocks or not 1 <= m.conv <= 16:
+                raise VoxB200Error(f"gated linear recurrence: {m.width} channels in {m.blocks} equal parts, convolution of 1 to 16 taps")
+        for m in ssm:
+            if m.heads % m.groups or m.inner % m.norm_groups or not 1 <= m.conv <= 16:
+                raise VoxB200Error(f"state space: {m.heads} heads in {m.groups} groups, {m.inner} channels in {m.norm_groups} norm groups, "
+                                   "convolution of 1 to 16 taps")
         self.x = torch.zeros(R, W, dtype=F32, device=dev)              # residual stream
         self.h = torch.zeros(R, W, dtype=CT, device=dev)               # normed input of the running sublayer
         self.y = torch.zeros(R, W, dtype=F32, device=dev)              # sublayer output
-        self.proj = torch.zeros(R * max(p_att + p_lin + p_lat + p_dif + p_gru + p_par + [1]), dtype=F32, device=dev)
+        self.proj = torch.zeros(R * max(p_att + p_lin + p_lat + p_dif + p_gru + p_par + p_ssm + p_pair + [1]), dtype=F32, device=dev)
         self.q = torch.zeros(R * max([m.heads * m.dim for m in att + lat] + [2 * m.heads * m.dim for m in dif] +
                                      [m.left.heads * m.left.dim for m in par] + [1]), dtype=CT, device=dev)
         for m in par:
@@ -973,8 +1127,18 @@ class HybridEngine:
             self.pair_o = torch.zeros(R * max(2 * m.heads * m.vdim for m in dif), dtype=F32, device=dev)   # both maps' outputs
         if gru:
             self.gru_scratch = None
+        if glr:
+            # the recurrence's input after its convolution, decays and scaled inputs of rows that it does not finish at once, the
+            # second mixer's output
+            self.glr_u = torch.zeros(R * max(m.width for m in glr), dtype=F32, device=dev)
+            self.glr_ab = torch.zeros(2 * R * max(m.width for m in glr), dtype=F32, device=dev)
+            self.y3 = torch.zeros(R, W, dtype=F32, device=dev)
+        if ssm:
+            self.ssm_x = torch.zeros(R * max(m.conv_channels for m in ssm), dtype=CT, device=dev)    # x | B | C after the convolution
+            self.ssm_o = torch.zeros(R * max(m.inner for m in ssm), dtype=F32, device=dev)           # gated output before its norm
         if cfg.block == "parallel":
-            self.h2 = torch.zeros(R, W, dtype=CT, device=dev)          # the feed-forward's norm of the same stream
+            if not cfg.shared_norm:
+                self.h2 = torch.zeros(R, W, dtype=CT, device=dev)      # the feed-forward's norm of the same stream
             self.y2 = torch.zeros(R, W, dtype=F32, device=dev)         # the feed-forward's output
         if lat:
             self.cq = torch.zeros(R * max(m.q_rank for m in lat), dtype=CT, device=dev)            # normed query latent
@@ -997,6 +1161,16 @@ class HybridEngine:
             n_t = max_rows // self.lin_tile_rows + max_out_rows + 1
             self.gru_scratch = torch.zeros(ops.mingru_scratch_floats(n_t, self.lin_tile_rows, max(m.width for m in gru))
                                            if dev.type == "cuda" else 1, dtype=F32, device=dev)
+        self.glr_scratch = self.ssm_scratch = None
+        if dev.type == "cuda":
+            n_t = max_rows // self.lin_tile_rows + cache.num_slots + 1
+            if glr:
+                self.glr_scratch = torch.zeros(ops.mingru_scratch_floats(n_t, self.lin_tile_rows, max(m.width for m in glr)), dtype=F32,
+                                               device=dev)
+            fits = [m for m in ssm if ops.ssd_tile_rows(m.vdim, m.state) == self.lin_tile_rows]
+            if fits:
+                self.ssm_scratch = torch.zeros(max(ops.ssd_scratch_floats(n_t, m.heads, m.vdim, m.state) for m in fits), dtype=F32,
+                                               device=dev)
         self.scan_scratch = None
         if par and dev.type == "cuda":
             n_t = max_rows // self.lin_tile_rows + cache.num_slots + 1
@@ -1077,7 +1251,7 @@ class HybridEngine:
     def _run_attention(self, s: StepInputs, q, kc, vc, out, gate, H: int, G: int, dim: int, vdim: int, window: int,
                        scale: float, head_rows: bool = False, **kw) -> None:
         """Prompt portions on the tiled kernel and single-token rows on the per-row kernel (split over keys with few rows).
-        kw: chunk, k_ld, v_ld, v_share of ``ops.window_attn``."""
+        kw: chunk, k_ld, v_ld, v_share, sink, keep_first, head_gate of ``ops.window_attn``."""
         tiles = None
         if s.tiles is not None and self.use_tiled_attention and vdim <= 256:
             tiles = (s.qo_indptr, s.tiles[0], s.tiles[1], s.tiles[2])
@@ -1127,10 +1301,15 @@ class HybridEngine:
         return self._proj(act, w["down"], out)
 
     def _attention(self, i: int, m: WindowAttentionConfig, w: Dict[str, Any], s: StepInputs) -> torch.Tensor:
-        T, W = s.T, self.cfg.width
-        nq, nk, nv = m.heads * m.dim, m.kv_heads * m.dim, m.kv_heads * m.vdim
-        P = nq + nk + nv + (m.heads * m.vdim if m.gate else 0)
+        T = s.T
+        P = m.heads * m.dim + m.kv_heads * (m.dim + m.vdim) + (0 if not m.gate else m.heads if m.head_gate else m.heads * m.vdim)
         proj = self._proj(self.h[:T], w["qkvg"], self.proj[:T * P].view(T, P))
+        return self._proj(self._attend(i, m, w, s, proj), w["o"], self.y[:T])
+
+    def _attend(self, i: int, m: WindowAttentionConfig, w: Dict[str, Any], s: StepInputs, proj: torch.Tensor) -> torch.Tensor:
+        """Projection rows [q | k | v (| gate) | ...] -> the concatenated (gated) heads: rotation and page append, attention."""
+        T = s.T
+        nq, nk, nv = m.heads * m.dim, m.kv_heads * m.dim, m.kv_heads * m.vdim
         cs, half, layout = None, 0, "half"
         if m.rotary is not None:
             cs, half, layout = self.cs[m.rotary.key()], m.rotary.dims // 2, m.rotary.layout
@@ -1147,8 +1326,8 @@ class HybridEngine:
         out = self.mix_out[:T * m.heads * m.vdim].view(T, m.heads * m.vdim)
         gate = proj[:, nq + nk + nv:] if m.gate else None
         self._run_attention(s, q, self.cache.k[i], self.cache.v[i], out, gate, m.heads, m.kv_heads, m.dim, m.vdim, m.window,
-                            m.scale, sink=w.get("sink"))
-        return self._proj(out, w["o"], self.y[:T])
+                            m.scale, sink=w.get("sink"), keep_first=m.keep_first, head_gate=m.head_gate)
+        return out
 
     def _lightning(self, i: int, m: DecayAttentionConfig, w: Dict[str, Any], s: StepInputs) -> torch.Tensor:
         T = s.T
@@ -1170,12 +1349,16 @@ class HybridEngine:
         return self._proj(out, w["o"], self.y[:T])
 
     def _moe_plain(self, f: MoEConfig, w: Dict[str, Any], s: StepInputs, h: torch.Tensor, out: torch.Tensor) -> torch.Tensor:
-        """Experts of the form down(act(up h)) behind the sigmoid router; the shared expert enters times its per-token gate."""
+        """Experts of the form down(act(up h)) behind the sigmoid router or a table over token ids; the shared expert enters times
+        its per-token gate."""
         T, W = s.T, self.cfg.width
         idx, wts = self.moe_idx[:T * f.top], self.moe_wts[:T * f.top]
         sgate = self.moe_sgate[:T] if (f.shared_ff and f.shared_gate) else None
-        ops.moe_route_sigmoid(h, w["router"], w.get("correction"), f.top, idx, wts, f.groups, f.groups_keep,
-                              w.get("sg") if sgate is not None else None, sgate)
+        sg = w.get("sg") if sgate is not None else None
+        if f.router == "table":
+            ops.moe_route_table(s.ids, w["table"], f.experts, idx, wts, h, sg, sgate)
+        else:
+            ops.moe_route_sigmoid(h, w["router"], w.get("correction"), f.top, idx, wts, f.groups, f.groups_keep, sg, sgate)
         if "grouped" in w and T >= self.GROUPED_MIN_ROWS:
             g, tt = w["grouped"], self.GROUP_TILE
             n_tiles = (T * f.top + tt - 1) // tt + f.experts
@@ -1290,7 +1473,7 @@ class HybridEngine:
         if T > self.max_rows or s.n_out > self.max_out_rows:
             raise VoxB200Error(f"step of {T} rows / {s.n_out} logit rows exceeds the engine's {self.max_rows} / {self.max_out_rows}")
         if cfg.block == "parallel":
-            return self._forward_parallel(s)
+            return self._forward_shared_norm(s) if cfg.shared_norm else self._forward_parallel(s)
         if cfg.block == "gated":
             return self._forward_gated(s)
         if cfg.block == "post":
@@ -1647,3 +1830,81 @@ class HybridEngine:
         # (a convolution of one tap keeps no inputs: any fp32 tensor stands in for its slot)
         ops.short_conv(h32, cw, None, state if state is not None else self.h32, s.qo_indptr, s.row_req, s.pos, s.slots, s.B, out=h,
                        residual=True)
+
+    # ---- parallel blocks with one shared norm --------------------------------------------------------------------
+    def _forward_shared_norm(self, s: StepInputs) -> torch.Tensor:
+        """x += mixer(h) + ff(h) with h = norm1(x) read by both sublayers.  The sum of a block's branches (a normed pair brings two,
+        each normed on the way) and the norm feeding the next block are one kernel (``ops.branch_residual_norm_f32``)."""
+        cfg, w, T = self.cfg, self.w, s.T
+        x, h, eps = self.x[:T], self.h[:T], cfg.eps
+        ops.embed_rows_f32(w.embed, s.ids, x, scale=cfg.embed_scale)
+        for key, freq in self.freqs.items():
+            ops.rotary_table(s.pos, freq, self.cs[key][:T], self.cs_mult[key])
+        n = len(cfg.layers)
+        if n:
+            ops.rmsnorm2_f32(x, w.layers[0]["norm1"], eps, h)
+        for i, L in enumerate(cfg.layers):
+            lw = w.layers[i]
+            if L.kind == "normed_pair":
+                branches = self._normed_pair(i, L.mixer, lw, s)
+            elif L.kind == "state_space":
+                branches = [(self._state_space(i, L.mixer, lw, s), None, cfg.residual_mult)]
+            else:
+                branches = [(self._attention(i, L.mixer, lw, s), None, cfg.residual_mult)]
+            if isinstance(L.mlp, DenseMLPConfig):
+                branches.append((self._dense_mlp(L.mlp, lw, h, self.y2[:T]), None, cfg.residual_mult))
+            elif L.mlp is not None:
+                branches.append((self._moe(L.mlp, lw, s, h=h, out=self.y2[:T]), None, cfg.residual_mult))
+            nxt = w.layers[i + 1]["norm1"] if i + 1 < n else None
+            ops.branch_residual_norm_f32(x, branches, eps, out=h if nxt is not None else None, w=nxt)
+            if self.layer_tap is not None:
+                self.layer_tap.append(x.clone())
+        return self._head(s)
+
+    def _normed_pair(self, i: int, m: NormedPairConfig, w: Dict[str, Any], s: StepInputs):
+        """Window attention and a gated linear recurrence side by side on one fused input projection -> the two outputs as
+        branches of the block's tail, which norms them."""
+        T, a, r = s.T, m.left, m.right
+        nqkv = a.heads * a.dim + a.kv_heads * (a.dim + a.vdim)
+        C = r.width
+        P = nqkv + 2 * C
+        proj = self._proj(self.h[:T], w["in"], self.proj[:T * P].view(T, P))
+        left = self._proj(self._attend(i, a, w, s, proj), w["left_o"], self.y[:T])
+        right = self._proj(self._gated_recurrence(i, r, w, s, proj[:, nqkv:nqkv + C], proj[:, nqkv + C:]), w["right_o"], self.y3[:T])
+        scale = m.scale * self.cfg.residual_mult
+        return [(left, w["left_norm"], scale), (right, w["right_norm"], scale)]
+
+    def _gated_recurrence(self, i: int, m: GatedLinearRecurrenceConfig, w: Dict[str, Any], s: StepInputs, y: torch.Tensor,
+                          x: torch.Tensor) -> torch.Tensor:
+        T, C, cache = s.T, m.width, self.cache
+        u = self.glr_u[:T * C].view(T, C)
+        ops.short_conv(x, w["conv"], w["conv_b"], cache.conv[(i, "x")], s.qo_indptr, s.row_req, s.pos, s.slots, s.B, out_f32=u,
+                       in_bias=w["x_b"])
+        out = self.mix_out[:T * C].view(T, C)
+        tiles = None
+        if (s.multi and s.tiles is not None and self.use_tiled_recurrence and
+                ops.mingru_scratch_floats(s.tiles[2], self.lin_tile_rows, C) <= self.glr_scratch.numel()):
+            tiles = (*s.tiles, self.lin_tile_rows)
+        return ops.rglru(u, w["gates"], w["gates_b"], w["lam"], m.c, y, w["y_b"], cache.state[i], out, self.glr_ab, s.qo_indptr, s.row_req,
+                         s.pos, s.slots, s.B, multi_rows=s.multi, tiles=tiles, scratch=self.glr_scratch)
+
+    def _state_space(self, i: int, m: StateSpaceConfig, w: Dict[str, Any], s: StepInputs) -> torch.Tensor:
+        T, inner, C, cache = s.T, m.inner, m.conv_channels, self.cache
+        P = inner + C + m.heads
+        proj = self._proj(self.h[:T], w["in"], self.proj[:T * P].view(T, P))
+        xbc = self.ssm_x[:T * C].view(T, C)
+        ops.short_conv(proj[:, inner:inner + C], w["conv"], w["conv_b"], cache.conv[(i, "x")], s.qo_indptr, s.row_req, s.pos, s.slots, s.B,
+                       out=xbc, act="silu")
+        o = self.ssm_o[:T * inner].view(T, inner)
+        args = (xbc, proj[:, inner + C:], w["dt_bias"], w["A_log"], w["D"], proj[:, :inner], cache.state[i], o, s.qo_indptr, s.pos, s.slots,
+                s.B, m.groups)
+        par = (s.multi and s.tiles is not None and self.use_tiled_recurrence and self.ssm_scratch is not None and
+               ops.ssd_tile_rows(m.vdim, m.state) == self.lin_tile_rows and
+               ops.ssd_scratch_floats(s.tiles[2], m.heads, m.vdim, m.state) <= self.ssm_scratch.numel())
+        if s.single or (s.multi and not par):
+            ops.ssd(*args, single_rows=s.single, multi_rows=s.multi and not par)
+        if par:
+            ops.ssd(*args, tiles=s.tiles, scratch=self.ssm_scratch)
+        out = self.mix_out[:T * inner].view(T, inner)
+        ops.group_rmsnorm(o, w["norm"], m.norm_groups, self.cfg.eps, out)
+        return self._proj(out, w["o"], self.y[:T])

@@ -1,7 +1,7 @@
 """Model-adapter registry with the reference's public surface (``vox_serve/model/__init__.py:17-179``):
 ``MODEL_REGISTRY``, ``get_model_class``, ``load_model``, ``register_model``, ``list_supported_models``.
 Only adapters whose whole decode + vocoder path runs on the sm_100a kernels are registered: Orpheus (+ SNAC) and CSM
-(+ Mimi) and Qwen3-TTS (+ its streaming 12 Hz codec decoder), and the text-only Bobavik, Razevik, Fovunex, Nadevik and Zopipel LMs.  A model given as a local
+(+ Mimi) and Qwen3-TTS (+ its streaming 12 Hz codec decoder), and the text-only Bobavik, Razevik, Fovunex, Nadevik, Zopipel and Redalix LMs.  A model given as a local
 directory is matched by the ``architecture`` of its ``config.json`` first, by its name otherwise."""
 from __future__ import annotations
 
@@ -20,6 +20,7 @@ from .nadevik import NadevikModel
 from .orpheus import OrpheusModel
 from .qwen3_tts import Qwen3TTSModel
 from .razevik import RazevikModel
+from .redalix import RedalixModel
 from .zopipel import ZopipelModel
 
 MODEL_REGISTRY: Dict[str, Type[BaseLM]] = {
@@ -34,6 +35,7 @@ MODEL_REGISTRY: Dict[str, Type[BaseLM]] = {
     "fovunex": FovunexModel,
     "nadevik": NadevikModel,
     "zopipel": ZopipelModel,
+    "redalix": RedalixModel,
 }
 
 

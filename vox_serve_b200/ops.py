@@ -923,7 +923,7 @@ def orpheus_window_codes(ids: torch.Tensor, audio_id_base: int):
 
 # ----------------------------------------------------------------------------------------------
 # hybrid decoder stacks with an fp32 residual stream (norm_linear.cu, window_attn.cu, linear_attn.cu, gated_recurrence.cu,
-# moe.cu)
+# ssd.cu, moe.cu)
 # dtype codes of the C ABI: 0 = bf16, 1 = fp32
 # ----------------------------------------------------------------------------------------------
 F32 = torch.float32
@@ -1218,6 +1218,105 @@ def mingru_tiled(proj: torch.Tensor, z_off: int, x_off: int, g_off: int, bz: Opt
     return out
 
 
+def rglru(u: torch.Tensor, w: torch.Tensor, bias: torch.Tensor, lam: torch.Tensor, c: float, y: torch.Tensor,
+          y_bias: Optional[torch.Tensor], state: torch.Tensor, out: torch.Tensor, ab: Optional[torch.Tensor], qo_indptr: torch.Tensor,
+          row_req: torch.Tensor, pos: torch.Tensor, slots: torch.Tensor, B: int, multi_rows: bool = True,
+          tiles: Optional[Tuple[torch.Tensor, torch.Tensor, int, int]] = None, scratch: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """Real-gated linear recurrent unit: r = sigmoid(R_b u + br), i = sigmoid(I_b u + bi) per block b of neighbouring channels,
+    log a = -c r softplus(lam), S_t = a S_(t-1) + sqrt(1 - a^2) i u, out = S * gelu_tanh(y + y_bias).  u, y: fp32 views [T, C];
+    w [blocks, 2 * C / blocks, C / blocks] (R_b above I_b; bf16 or fp32), bias fp32 [blocks, 2 * C / blocks]; state fp32
+    [slots, C] (taken as zero where a request starts at position 0); out a view [T, C] (bf16 or fp32).  multi_rows: some request
+    brings several rows (ab: fp32 scratch of 2 T C); tiles = (tile_req, tile_row0, n_tiles, tile_rows) + scratch: those in
+    parallel pieces instead of row by row."""
+    _need_cuda(u, w, y, state, out)
+    T, C = u.shape
+    blocks, bs = w.shape[0], w.shape[2]
+    assert u.dtype == F32 and u.stride(1) == 1 and y.dtype == F32 and y.stride(1) == 1 and tuple(y.shape) == (T, C)
+    assert w.is_contiguous() and w.shape[1] == 2 * bs and blocks * bs == C and bias.dtype == F32 and bias.numel() == 2 * C
+    assert lam.dtype == F32 and lam.numel() == C and (y_bias is None or (y_bias.dtype == F32 and y_bias.numel() == C))
+    assert state.dtype == F32 and state.is_contiguous() and state.shape[1] == C and out.stride(1) == 1 and tuple(out.shape) == (T, C)
+    assert not multi_rows or (ab is not None and ab.dtype == F32 and ab.numel() >= 2 * T * C)
+    tr = t0 = None
+    n_tiles = tile_rows = 0
+    if multi_rows and tiles is not None:
+        tile_req, tile_row0, n_tiles, tile_rows = tiles
+        tr, t0 = tile_req.data_ptr(), tile_row0.data_ptr()
+        assert scratch is not None and scratch.dtype == F32 and scratch.numel() >= mingru_scratch_floats(n_tiles, tile_rows, C)
+    call("vb_rglru", out.data_ptr(), out.stride(0), state.data_ptr(), _p(ab), _p(scratch), u.data_ptr(), u.stride(0), w.data_ptr(),
+         bias.data_ptr(), lam.data_ptr(), float(c), y.data_ptr(), y.stride(0), _p(y_bias), qo_indptr.data_ptr(), row_req.data_ptr(),
+         pos.data_ptr(), slots.data_ptr(), tr, t0, n_tiles, tile_rows, T, B, C, blocks, int(multi_rows), _dt(w), _dt(out), _stream())
+    if multi_rows:
+        _lib.launch_counter[0] += 3 if n_tiles else 1      # (beside the one that ``call`` counts)
+    return out
+
+
+def ssd_tile_rows(vdim: int, states: int) -> int:
+    return _lib.load().vb_ssd_tile_rows(int(vdim), int(states))
+
+
+def ssd_scratch_floats(n_tiles: int, heads: int, vdim: int, states: int) -> int:
+    return _lib.load().vb_ssd_scratch_floats(int(n_tiles), int(heads), int(vdim), int(states))
+
+
+def ssd(xbc: torch.Tensor, dt: torch.Tensor, dt_bias: torch.Tensor, A_log: torch.Tensor, D: torch.Tensor, z: torch.Tensor,
+        state: torch.Tensor, out: torch.Tensor, qo_indptr: torch.Tensor, pos: torch.Tensor, slots: torch.Tensor, B: int, groups: int,
+        single_rows: bool = True, multi_rows: bool = True, tiles: Optional[Tuple[torch.Tensor, torch.Tensor, int]] = None,
+        scratch: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """dt = softplus(dt + dt_bias);  S_t = exp(-exp(A_log) dt) S_(t-1) + dt B_t x_t^T;  y = S^T C + D x;  out = y * silu(z), per
+    head.  xbc [T, H V + 2 G N] (bf16 or fp32; x | B | C, heads in order share their group's B and C); dt an fp32 view [T, H], z
+    one [T, H V]; state fp32 [slots, H, N, V] (taken as zero where a request starts at position 0); out fp32 [T, H V].
+    tiles = (tile_req, tile_row0, n_tiles) + scratch: prompt portions as parallel tiles of ``ssd_tile_rows`` rows (requests that
+    bring one row are then left to a second call)."""
+    _need_cuda(xbc, dt, z, state, out)
+    _, H, N, V = state.shape
+    T = xbc.shape[0]
+    assert xbc.stride(1) == 1 and xbc.shape[1] == H * V + 2 * groups * N and out.dtype == F32 and out.is_contiguous()
+    assert dt.dtype == F32 and dt.stride(1) == 1 and dt.shape[1] == H and z.dtype == F32 and z.stride(1) == 1 and z.shape[1] == H * V
+    assert state.dtype == F32 and state.is_contiguous() and tuple(out.shape) == (T, H * V)
+    for v in (dt_bias, A_log, D):
+        assert v.dtype == F32 and v.numel() == H
+    head = (out.data_ptr(), state.data_ptr())
+    body = (xbc.data_ptr(), xbc.stride(0), dt.data_ptr(), dt.stride(0), dt_bias.data_ptr(), A_log.data_ptr(), D.data_ptr(),
+            z.data_ptr(), z.stride(0), qo_indptr.data_ptr(), pos.data_ptr(), slots.data_ptr())
+    if tiles is None:
+        call("vb_ssd", *head, *body, B, H, V, N, groups, int(single_rows), int(multi_rows), _dt(xbc), _stream())
+    else:
+        tile_req, tile_row0, n_tiles = tiles
+        assert scratch is not None and scratch.dtype == F32 and scratch.numel() >= ssd_scratch_floats(n_tiles, H, V, N)
+        call("vb_ssd_tiled", *head, scratch.data_ptr(), *body, tile_req.data_ptr(), tile_row0.data_ptr(), n_tiles, B, H, V, N, groups,
+             _dt(xbc), _stream())
+    return out
+
+
+def group_rmsnorm(x: torch.Tensor, w: torch.Tensor, groups: int, eps: float, out: torch.Tensor) -> torch.Tensor:
+    """out (bf16 or fp32) = rows of x (fp32 [T, C]) in ``groups`` equal neighbourhoods of channels, each divided by its own root mean
+    square, times w (fp32 [C])."""
+    _need_cuda(x, w, out)
+    assert x.dtype == F32 and x.is_contiguous() and out.is_contiguous() and tuple(out.shape) == tuple(x.shape)
+    assert w.dtype == F32 and w.numel() == x.shape[1] and x.shape[1] % groups == 0
+    call("vb_group_rmsnorm", out.data_ptr(), x.data_ptr(), w.data_ptr(), x.shape[0], x.shape[1], int(groups), float(eps), _dt(out),
+         _stream())
+    return out
+
+
+def branch_residual_norm_f32(x: torch.Tensor, branches, eps: float, out: Optional[torch.Tensor] = None,
+                             w: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """x += sum over branches (y, norm weight or None, scale) of scale * (y / rms(y) * weight, or y itself) in place (fp32
+    [T, W], at most three branches); out (bf16 or fp32, optional) = the new x / rms(x) * w."""
+    _need_cuda(x)
+    assert x.dtype == F32 and x.is_contiguous() and 1 <= len(branches) <= 3
+    args = []
+    for k in range(3):
+        y, wk, scale = branches[k] if k < len(branches) else (None, None, 0.0)
+        assert y is None or (y.dtype == F32 and y.is_contiguous() and tuple(y.shape) == tuple(x.shape))
+        assert wk is None or (wk.dtype == F32 and wk.numel() == x.shape[1])
+        args += [_p(y), _p(wk), float(scale)]
+    assert out is None or (w is not None and out.is_contiguous() and tuple(out.shape) == tuple(x.shape))
+    call("vb_branch_residual_norm_f32", x.data_ptr(), *args, _p(out), _p(w) if out is not None else None, x.shape[0], x.shape[1],
+         float(eps), _dt(out) if out is not None else 1, _stream())
+    return x
+
+
 def qkv_rotary_append(proj: torch.Tensor, q_off: int, k_off: int, v_off: int, cs: Optional[torch.Tensor], half: int,
                       q_out: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor, row_req: torch.Tensor,
                       pos: torch.Tensor, page_indptr: torch.Tensor, page_indices: torch.Tensor, T: int, H: int, G: int,
@@ -1237,7 +1336,7 @@ def window_attn(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor, o
                 tiles: Optional[Tuple[torch.Tensor, torch.Tensor, torch.Tensor, int]] = None,
                 scratch: Optional[torch.Tensor] = None, rows: Optional[Tuple[torch.Tensor, int]] = None,
                 head_rows: bool = False, chunk: int = 0, k_ld: int = 0, v_ld: int = 0, v_share: int = 1,
-                sink: Optional[torch.Tensor] = None) -> torch.Tensor:
+                sink: Optional[torch.Tensor] = None, keep_first: int = 0, head_gate: bool = False) -> torch.Tensor:
     """gate: an fp32 view [T, H * vdim] (any row stride) or None.  tiles = (qo_indptr, tile_req, tile_row0, n_tiles):
     run the tiled prompt kernel over those row tiles instead of the per-row kernel.  scratch (fp32): lets the per-row kernel
     split a row's keys over several CTAs when the step has few rows.  rows = (int32 row indices, count): serve only those
@@ -1246,7 +1345,8 @@ def window_attn(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor, o
     only the keys of its own block of `chunk` positions.  k_ld / v_ld: elements per token of the key / value cache when they
     are not G * dim / G * vdim (values that are a leading slice of the key rows).  v_share: consecutive key heads reading one
     value head.  An fp32 ``out`` beside bf16 operands is written in fp32.  sink (fp32 [H]): exp(sink[h]) joins the denominator of
-    head h's softmax."""
+    head h's softmax.  keep_first: the first so many positions are visible to every later one, however far.  head_gate: the gate
+    holds one value per head ([T, H]) instead of one per output value."""
     _need_cuda(q, k_cache, v_cache, out)
     assert sink is None or (sink.dtype == F32 and sink.numel() == H)
     out_f32 = int(out.dtype == F32)
@@ -1257,13 +1357,13 @@ def window_attn(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor, o
              row_req.data_ptr(), pos.data_ptr(), page_indptr.data_ptr(), page_indices.data_ptr(), n, H, G, dim, vdim,
              k_cache.shape[1], int(window), float(scale), _dt(q), _p(scratch), scratch.numel() if scratch is not None else 0,
              _p(rows[0]) if rows is not None else None, int(head_rows), int(chunk), int(k_ld), int(v_ld), int(v_share), out_f32,
-             _p(sink), _stream())
+             _p(sink), int(keep_first), int(head_gate), _stream())
     else:
         qo, tile_req, tile_row0, n_tiles = tiles
         call("vb_window_attn_tiled", out.data_ptr(), q.data_ptr(), k_cache.data_ptr(), v_cache.data_ptr(), _p(gate),
              ld_gate, pos.data_ptr(), page_indptr.data_ptr(), page_indices.data_ptr(), qo.data_ptr(), tile_req.data_ptr(),
              tile_row0.data_ptr(), n_tiles, T, H, G, dim, vdim, k_cache.shape[1], int(window), float(scale), _dt(q),
-             int(chunk), int(k_ld), int(v_ld), int(v_share), out_f32, _p(sink), _stream())
+             int(chunk), int(k_ld), int(v_ld), int(v_share), out_f32, _p(sink), int(keep_first), int(head_gate), _stream())
     return out
 
 
@@ -1332,6 +1432,19 @@ def moe_route_sigmoid(h: torch.Tensor, router_w: torch.Tensor, correction: Optio
     call("vb_moe_route_sigmoid", idx.data_ptr(), wts.data_ptr(), _p(shared_gate), h.data_ptr(), router_w.data_ptr(),
          _p(correction), _p(shared_gate_w), h.shape[0], h.shape[1], router_w.shape[0], top, int(groups), int(keep), _dt(h),
          _stream())
+
+
+def moe_route_table(ids: torch.Tensor, table: torch.Tensor, experts: int, idx: torch.Tensor, wts: torch.Tensor,
+                    h: Optional[torch.Tensor] = None, shared_gate_w: Optional[torch.Tensor] = None,
+                    shared_gate: Optional[torch.Tensor] = None) -> None:
+    """idx[t] = table[ids[t]] (int32 [vocab, top]), every weight 1 / top; shared_gate (fp32 [T], optional) =
+    sigmoid(shared_gate_w . h)."""
+    _need_cuda(ids, table, idx, wts)
+    assert ids.dtype == table.dtype == idx.dtype == torch.int32 and table.is_contiguous() and wts.dtype == F32
+    assert shared_gate_w is None or (shared_gate_w.dtype == F32 and h.is_contiguous() and shared_gate_w.numel() == h.shape[1])
+    call("vb_moe_route_table", idx.data_ptr(), wts.data_ptr(), _p(shared_gate), ids.data_ptr(), table.data_ptr(), _p(h),
+         _p(shared_gate_w), ids.numel(), h.shape[1] if h is not None else 0, table.shape[0], int(experts), table.shape[1],
+         _dt(h) if h is not None else 1, _stream())
 
 
 def moe_group(idx: torch.Tensor, T: int, experts: int, top: int, row_off: torch.Tensor, sorted_token: torch.Tensor,
@@ -1432,24 +1545,27 @@ def pair_hash_rows(rows: torch.Tensor, prev_tok: torch.Tensor, ids: torch.Tensor
 
 def short_conv(x: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor], state: torch.Tensor, qo_indptr: torch.Tensor,
                row_req: torch.Tensor, pos: torch.Tensor, slots: torch.Tensor, B: int, out: Optional[torch.Tensor] = None,
-               out_f32: Optional[torch.Tensor] = None, act: Optional[str] = None, residual: bool = False) -> None:
+               out_f32: Optional[torch.Tensor] = None, act: Optional[str] = None, residual: bool = False,
+               in_bias: Optional[torch.Tensor] = None) -> None:
     """Causal convolution over time on every channel of x (an fp32 view [T, C], any row stride): y_t = bias + sum_j w[:, j]
     x_(t - taps + 1 + j), zeros before a request's start; w fp32 [C, taps]; act "silu" or None; residual: x_t is added to the
-    result.  state fp32 [slots, taps - 1, C]: a request's last inputs, read by the step's first rows and advanced by the step.
+    result; in_bias fp32 [C] is added to every input row first (the zeros before the start stay zero).  state fp32
+    [slots, taps - 1, C]: a request's last inputs (bias included), read by the step's first rows and advanced by the step.
     out (bf16 or fp32 view [T, C]) and / or out_f32 (fp32 view) receive the result."""
     _need_cuda(x, w, state)
     T, C = x.shape
     taps = w.shape[1]
     assert x.dtype == F32 and x.stride(1) == 1 and w.dtype == F32 and w.is_contiguous() and w.shape[0] == C
     assert state.dtype == F32 and state.is_contiguous() and (taps == 1 or tuple(state.shape[1:]) == (taps - 1, C))
-    assert bias is None or (bias.dtype == F32 and bias.numel() == C)
+    for v in (bias, in_bias):
+        assert v is None or (v.dtype == F32 and v.numel() == C)
     for o in (out, out_f32):
         assert o is None or (o.stride(1) == 1 and tuple(o.shape) == (T, C))
     assert out_f32 is None or out_f32.dtype == F32
     call("vb_short_conv", _p(out), out.stride(0) if out is not None else 0, _p(out_f32),
          out_f32.stride(0) if out_f32 is not None else 0, x.data_ptr(), x.stride(0), w.data_ptr(), _p(bias), state.data_ptr(),
          qo_indptr.data_ptr(), row_req.data_ptr(), pos.data_ptr(), slots.data_ptr(), T, B, C, taps, 1 if act == "silu" else 0,
-         int(residual), _dt(out) if out is not None else 1, _stream())
+         int(residual), _dt(out) if out is not None else 1, _p(in_bias), _stream())
 
 
 HYPER_CONV_TAPS = 4        # the longest convolution that hyper_mix_norm runs by itself

@@ -1,5 +1,5 @@
 """Worker for text-only LMs on the hybrid engine (model/bobavik.py, model/razevik.py, model/fovunex.py, model/nadevik.py,
-model/zopipel.py): the same five scheduler-facing methods, page pool, batch slots, packed staging buffer, sampled-id ring and
+model/zopipel.py, model/redalix.py): the same five scheduler-facing methods, page pool, batch slots, packed staging buffer, sampled-id ring and
 decode CUDA graphs as ``ModelWorker``, with three differences.
 
   * Prompts are fed in portions.  A request carries ``pending_tokens`` (the rest of its prompt, or continuation tokens a
