@@ -23,6 +23,12 @@ softmax sink; gated gelu feed-forward) beside its closest relative on the same e
 rotated key part, gated residuals, gated dense feed-forward) with as many latent-attention and softmax-attention layers, at equal
 width, head count, head size and feed-forward width -- and beside Bobavik with attention layers only.
 
+``--arch redalix``: the Redalix design (parallel blocks on one shared norm; window attention with kept first tokens and a sink beside
+a real-gated linear recurrent unit, attention with biases and a gate per head, Mamba-2; table-routed squared-relu experts and a gated
+shared expert) beside its closest relatives on the same engine, Nadevik (attention beside a selective scan, mixture of experts) and
+Bobavik (window attention, linear attention with a recurrent state, mixture of experts), at equal width, head count, head size and
+expert width per token.
+
 Per size and engine: prefill of one 1024-token prompt (eager launches) and one decode step of 32 requests at context 512
 (a CUDA-graph replay, as served), timed with CUDA events after warm-up; an L2-sized buffer is overwritten between timed
 iterations.  Output: one JSON line per size.
@@ -111,6 +117,23 @@ def zopipel_config(width: int, ff: int) -> dict:
             "layers": layers}
 
 
+def redalix_config(width: int, ff: int, experts: int = 8, top: int = 2) -> dict:
+    """four layers: Mamba-2, mixer pair, attention, mixer pair, each with experts (8, top 2, and a shared one: the expert width a
+    Bobavik token uses).  128-wide heads, a quarter as many key/value heads (pair: window 2048 and 4 kept tokens; attention: window
+    4096, rotated whole with YaRN scaling); recurrence as wide as the model in blocks of 256; Mamba-2: twice the width in heads of
+    64, 128 states, 8 groups; convolutions of 4 taps"""
+    heads = width // 128
+    att = {"heads": heads, "kv_heads": max(1, heads // 4), "dim": 128, "vdim": 128, "scale": 128 ** -0.5}
+    pair = {"left": dict(att, mask={"size": 2048, "keep_first": 4}), "right": {"width": width, "blocks": width // 256, "conv": 4}}
+    rot = {"dims": 128, "base": 1e6, "scaling": {"factor": 4.0, "original": 8192, "fast": 32.0, "slow": 1.0}}
+    ssm = {"heads": width // 32, "vdim": 64, "state": 128, "groups": 8, "norm_groups": 8, "conv": 4}
+    mlp = {"kind": "moe", "router": {"experts": experts, "top": top}, "expert": {"ff": ff}, "shared": {"ff": ff}}
+    layers = [{"type": "mamba2", "mixer": ssm, "mlp": dict(mlp)}, {"type": "parallel", "mixer": dict(pair), "mlp": dict(mlp)},
+              {"type": "attention", "mixer": dict(att, mask={"size": 4096}, rot=rot), "mlp": dict(mlp)},
+              {"type": "parallel", "mixer": dict(pair), "mlp": dict(mlp)}]
+    return {"architecture": "Redalix", "width": width, "vocab": VOCAB, "norm": {"eps": 1e-6}, "layers": layers}
+
+
 def fovunex_attention_config(width: int, ff: int) -> dict:
     """Fovunex as Zopipel's neighbour: latent attention, two-map attention, two-map attention, latent attention, each with a
     feed-forward (the two maps of 64 dims make 128 query / key dims per head)"""
@@ -169,9 +192,12 @@ def bench_bobavik(width: int, ff: int, steps: int, warmup: int, flush, kinds=Non
     from vox_serve_b200.model.fovunex import FovunexModel
     from vox_serve_b200.model.nadevik import NadevikModel
     from vox_serve_b200.model.razevik import RazevikModel
+    from vox_serve_b200.model.redalix import RedalixModel
     from vox_serve_b200.model.zopipel import ZopipelModel
 
-    if design == "zopipel":
+    if design == "redalix":
+        model = RedalixModel("redalix-synthetic:1", config=redalix_config(width, ff), device="cuda:0")
+    elif design == "zopipel":
         model = ZopipelModel("zopipel-synthetic:1", config=zopipel_config(width, ff), device="cuda:0")
     elif design == "fovunex_attention":
         model = FovunexModel("fovunex-synthetic:1", config=fovunex_attention_config(width, ff), device="cuda:0")
@@ -266,62 +292,32 @@ def bench_llama(width: int, inter: int, steps: int, warmup: int, flush) -> dict:
             "decode_tok_s": BATCH / t_dec * 1e3, "weight_gb": w.nbytes() / 1e9}
 
 
+# --arch -> (name of the comparison, the sides: key of the output line, --arch-only name, what runs)
+COMPARISONS = {
+    "bobavik": ("bobavik_vs_llama", (("bobavik", "bobavik", {}), ("llama", "llama", None))),
+    "razevik": ("razevik_vs_bobavik_attention", (("razevik", "razevik", {"design": "razevik"}),
+                                                 ("bobavik_attention", "bobavik", {"kinds": ("attention",) * LAYERS}))),
+    "fovunex": ("fovunex_vs_bobavik", (("fovunex", "fovunex", {"design": "fovunex"}), ("bobavik", "bobavik", {}))),
+    "nadevik": ("nadevik_vs_bobavik", (("nadevik", "nadevik", {"design": "nadevik"}), ("bobavik", "bobavik", {}))),
+    "zopipel": ("zopipel_vs_fovunex", (("zopipel", "zopipel", {"design": "zopipel"}),
+                                       ("fovunex", "fovunex", {"design": "fovunex_attention"}),
+                                       ("bobavik_attention", "bobavik", {"kinds": ("attention",) * LAYERS}))),
+    "redalix": ("redalix_vs_nadevik", (("redalix", "redalix", {"design": "redalix"}), ("nadevik", "nadevik", {"design": "nadevik"}),
+                                       ("bobavik", "bobavik", {}))),
+}
+
+
 def run(sizes, steps: int, warmup: int, only: str = "", arch: str = "bobavik") -> None:
     flush = torch.zeros(192 << 20, dtype=torch.uint8, device="cuda")
+    name, sides = COMPARISONS[arch]
     for width in sizes:
         ff = width                     # expert width; a token uses top (2) experts + the shared one
-        if arch == "fovunex":
-            line = {"bench": "fovunex_vs_bobavik", "width": width, "layers": LAYERS, "prompt": PROMPT, "decode_batch": BATCH,
-                    "context": CONTEXT, "steps": steps, "warmup": warmup, "dtype": "bf16", "data": "synthetic",
-                    "l2": "192 MiB buffer overwritten between timed iterations"}
-            if only in ("", "fovunex"):
-                line["fovunex"] = bench_bobavik(width, ff, steps, warmup, flush, design="fovunex")
-            if only in ("", "bobavik"):
-                line["bobavik"] = bench_bobavik(width, ff, steps, warmup, flush)
-            print(json.dumps(line), flush=True)
-            torch.cuda.empty_cache()
-            continue
-        if arch == "zopipel":
-            line = {"bench": "zopipel_vs_fovunex", "width": width, "layers": LAYERS, "prompt": PROMPT, "decode_batch": BATCH,
-                    "context": CONTEXT, "steps": steps, "warmup": warmup, "dtype": "bf16", "data": "synthetic",
-                    "l2": "192 MiB buffer overwritten between timed iterations"}
-            if only in ("", "zopipel"):
-                line["zopipel"] = bench_bobavik(width, ff, steps, warmup, flush, design="zopipel")
-            if only in ("", "fovunex"):
-                line["fovunex"] = bench_bobavik(width, ff, steps, warmup, flush, design="fovunex_attention")
-            if only in ("", "bobavik"):
-                line["bobavik_attention"] = bench_bobavik(width, ff, steps, warmup, flush, kinds=("attention",) * LAYERS)
-            print(json.dumps(line), flush=True)
-            torch.cuda.empty_cache()
-            continue
-        if arch == "nadevik":
-            line = {"bench": "nadevik_vs_bobavik", "width": width, "layers": LAYERS, "prompt": PROMPT, "decode_batch": BATCH,
-                    "context": CONTEXT, "steps": steps, "warmup": warmup, "dtype": "bf16", "data": "synthetic",
-                    "l2": "192 MiB buffer overwritten between timed iterations"}
-            if only in ("", "nadevik"):
-                line["nadevik"] = bench_bobavik(width, ff, steps, warmup, flush, design="nadevik")
-            if only in ("", "bobavik"):
-                line["bobavik"] = bench_bobavik(width, ff, steps, warmup, flush)
-            print(json.dumps(line), flush=True)
-            torch.cuda.empty_cache()
-            continue
-        if arch == "razevik":
-            line = {"bench": "razevik_vs_bobavik_attention", "width": width, "layers": LAYERS, "prompt": PROMPT,
-                    "decode_batch": BATCH, "context": CONTEXT, "steps": steps, "warmup": warmup, "dtype": "bf16",
-                    "data": "synthetic", "l2": "192 MiB buffer overwritten between timed iterations"}
-            if only in ("", "razevik"):
-                line["razevik"] = bench_bobavik(width, ff, steps, warmup, flush, design="razevik")
-            if only in ("", "bobavik"):
-                line["bobavik_attention"] = bench_bobavik(width, ff, steps, warmup, flush, kinds=("attention",) * LAYERS)
-            print(json.dumps(line), flush=True)
-            torch.cuda.empty_cache()
-            continue
-        line = {"bench": "bobavik_vs_llama", "width": width, "layers": LAYERS, "prompt": PROMPT, "decode_batch": BATCH,
-                "context": CONTEXT, "steps": steps, "warmup": warmup, "dtype": "bf16", "data": "synthetic",
+        line = {"bench": name, "width": width, "layers": LAYERS, "prompt": PROMPT, "decode_batch": BATCH, "context": CONTEXT,
+                "steps": steps, "warmup": warmup, "dtype": "bf16", "data": "synthetic",
                 "l2": "192 MiB buffer overwritten between timed iterations"}
-        if only in ("", "bobavik"):
-            line["bobavik"] = bench_bobavik(width, ff, steps, warmup, flush)
-        if only in ("", "llama"):
-            line["llama"] = bench_llama(width, 3 * ff, steps, warmup, flush)
+        for key, side, kw in sides:
+            if only in ("", side):
+                line[key] = (bench_llama(width, 3 * ff, steps, warmup, flush) if kw is None
+                             else bench_bobavik(width, ff, steps, warmup, flush, **kw))
         print(json.dumps(line), flush=True)
         torch.cuda.empty_cache()

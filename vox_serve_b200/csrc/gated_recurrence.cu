@@ -141,17 +141,17 @@ __global__ void __launch_bounds__(128) mingru_tile_scan_kernel(MinGruParams p) {
   float S = p.pos[r0] == 0 ? 0.f : *st;
   float* s = p.scratch + static_cast<size_t>(lo) * ppt * 2 * p.width + ch;
   const int n = (last - lo) * ppt;
-  // (the summaries do not depend on S: eight pieces' loads are issued before their chain runs)
-  for (int i0 = 0; i0 < n; i0 += 8) {
-    float A[8], Bv[8];
+  // (the summaries do not depend on S: sixteen pieces' loads are issued before their chain runs)
+  for (int i0 = 0; i0 < n; i0 += 16) {
+    float A[16], Bv[16];
 #pragma unroll
-    for (int i = 0; i < 8; ++i) {
+    for (int i = 0; i < 16; ++i) {
       const bool ok = i0 + i < n;
       A[i] = ok ? s[static_cast<size_t>(i0 + i) * 2 * p.width] : 1.f;
       Bv[i] = ok ? s[static_cast<size_t>(i0 + i) * 2 * p.width + p.width] : 0.f;
     }
 #pragma unroll
-    for (int i = 0; i < 8; ++i) {
+    for (int i = 0; i < 16; ++i) {
       if (i0 + i < n) {
         s[static_cast<size_t>(i0 + i) * 2 * p.width] = S;
         S = A[i] * S + Bv[i];
@@ -302,6 +302,147 @@ __global__ void __launch_bounds__(256) rglru_gates_kernel(RgLruParams p) {
   }
 }
 
+// bf16 matrices, blocks of a multiple of 16 channels: CTA = 64 rows x 32 channels of one block (64 gate columns: r, then i), 4
+// warps x 16 rows, mma.sync m16n8k16 with fp32 accumulators over chunks of 64 inputs; u enters as two bf16 terms (its rounding
+// and the remainder's).  The next chunk's loads are in flight while a chunk is multiplied.
+constexpr int RM_R = 64, RM_CH = 32, RM_K = 64, RM_LD = RM_K + 8;
+
+template <typename CT>
+__global__ void __launch_bounds__(128) rglru_gates_mma_kernel(RgLruParams p) {
+  __shared__ __align__(16) __nv_bfloat16 Uh[RM_R * RM_LD], Ul[RM_R * RM_LD], Ws[2 * RM_CH * RM_LD];
+  const int per = (p.bs + RM_CH - 1) / RM_CH, blk = blockIdx.x / per, c0 = (blockIdx.x - blk * per) * RM_CH;
+  const int t0 = blockIdx.y * RM_R, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  const __nv_bfloat16* W = static_cast<const __nv_bfloat16*>(p.w) + static_cast<size_t>(blk) * 2 * p.bs * p.bs;
+  const int ur = tid >> 4, uc = (tid & 15) * 4, wr = tid >> 3, wc = (tid & 7) * 8;
+  float4 un[8];
+  uint4 wn[4];
+  auto fetch_w = [&](int k0) {
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+      const int r = wr + 16 * i, ch = c0 + (r & (RM_CH - 1));
+      wn[i] = make_uint4(0u, 0u, 0u, 0u);
+      if (ch < p.bs && k0 + wc < p.bs)
+        wn[i] = *reinterpret_cast<const uint4*>(W + static_cast<size_t>((r >= RM_CH ? p.bs : 0) + ch) * p.bs + k0 + wc);
+    }
+  };
+  auto fetch_u = [&](int k0) {
+#pragma unroll
+    for (int i = 0; i < 8; ++i) {
+      const int t = t0 + ur + 8 * i;
+      un[i] = make_float4(0.f, 0.f, 0.f, 0.f);
+      if (t < p.T && k0 + uc < p.bs) un[i] = *reinterpret_cast<const float4*>(p.u + static_cast<size_t>(t) * p.ld_u + blk * p.bs + k0 + uc);
+    }
+  };
+  fetch_w(0);                             // (weights: nothing that precedes this launch writes them)
+  pdl_sync();
+  fetch_u(0);
+  float acc[8][4];
+#pragma unroll
+  for (int n = 0; n < 8; ++n) acc[n][0] = acc[n][1] = acc[n][2] = acc[n][3] = 0.f;
+  const bool rows = t0 + warp * 16 < p.T;
+  for (int k0 = 0; k0 < p.bs; k0 += RM_K) {
+#pragma unroll
+    for (int i = 0; i < 8; ++i) {
+      const float v[4] = {un[i].x, un[i].y, un[i].z, un[i].w};
+      float hi[4], lo[4];
+#pragma unroll
+      for (int e = 0; e < 4; ++e) {
+        hi[e] = __bfloat162float(__float2bfloat16_rn(v[e]));
+        lo[e] = v[e] - hi[e];
+      }
+      const int o = (ur + 8 * i) * RM_LD + uc;
+      *reinterpret_cast<uint2*>(Uh + o) = make_uint2(pack_bf16(hi[0], hi[1]), pack_bf16(hi[2], hi[3]));
+      *reinterpret_cast<uint2*>(Ul + o) = make_uint2(pack_bf16(lo[0], lo[1]), pack_bf16(lo[2], lo[3]));
+    }
+#pragma unroll
+    for (int i = 0; i < 4; ++i) *reinterpret_cast<uint4*>(Ws + (wr + 16 * i) * RM_LD + wc) = wn[i];
+    __syncthreads();
+    if (k0 + RM_K < p.bs) {
+      fetch_w(k0 + RM_K);
+      fetch_u(k0 + RM_K);
+    }
+    if (rows) {
+#pragma unroll
+      for (int kb = 0; kb < RM_K / 16; ++kb) {
+        if (k0 + kb * 16 < p.bs) {
+          const int ao = (warp * 16 + (lane & 15)) * RM_LD + kb * 16 + (lane >> 4) * 8;
+          uint32_t ah[4], al[4];
+          ldmatrix_x4(ah, smem_u32(Uh + ao));
+          ldmatrix_x4(al, smem_u32(Ul + ao));
+#pragma unroll
+          for (int np = 0; np < 4; ++np) {
+            uint32_t bf[4];
+            ldmatrix_x4(bf, smem_u32(Ws + (np * 16 + (lane >> 4) * 8 + (lane & 7)) * RM_LD + kb * 16 + ((lane >> 3) & 1) * 8));
+            mma_bf16_16816(acc[2 * np], ah, bf[0], bf[1]);
+            mma_bf16_16816(acc[2 * np], al, bf[0], bf[1]);
+            mma_bf16_16816(acc[2 * np + 1], ah, bf[2], bf[3]);
+            mma_bf16_16816(acc[2 * np + 1], al, bf[2], bf[3]);
+          }
+        }
+      }
+    }
+    __syncthreads();
+  }
+  if (!rows) return;
+  // as rg_finish, with all loads of a row's eight channels in flight before the first store
+  const int lc = c0 + (lane & 3) * 2, gc = blk * p.bs + lc;
+  const float* bias = p.bias + static_cast<size_t>(blk) * 2 * p.bs + lc;
+  float lam[4][2], br[4][2], bi[4][2];
+#pragma unroll
+  for (int n = 0; n < 4; ++n)
+#pragma unroll
+    for (int e = 0; e < 2; ++e) {
+      const bool ok = lc + n * 8 < p.bs;
+      lam[n][e] = ok ? p.lam[gc + n * 8 + e] : 0.f;
+      br[n][e] = ok ? bias[n * 8 + e] : 0.f;
+      bi[n][e] = ok ? bias[p.bs + n * 8 + e] : 0.f;
+    }
+#pragma unroll
+  for (int half = 0; half < 2; ++half) {
+    const int t = t0 + warp * 16 + (lane >> 2) + 8 * half;
+    if (t >= p.T) continue;
+    const int b = p.row_req[t];
+    const bool single = p.qo_indptr[b + 1] - p.qo_indptr[b] == 1, fresh = p.pos[t] == 0;
+    float* st = p.state + static_cast<size_t>(p.slots[b]) * p.C + gc;
+    const float* yr = p.y + static_cast<size_t>(t) * p.ld_y + gc;
+    float2 u[4];
+    float S[4][2], y[4][2];
+#pragma unroll
+    for (int n = 0; n < 4; ++n) {
+      const bool ok = lc + n * 8 < p.bs;
+      u[n] = ok ? *reinterpret_cast<const float2*>(p.u + static_cast<size_t>(t) * p.ld_u + gc + n * 8) : make_float2(0.f, 0.f);
+#pragma unroll
+      for (int e = 0; e < 2; ++e) {
+        S[n][e] = ok && single && !fresh ? st[n * 8 + e] : 0.f;
+        y[n][e] = ok && single ? yr[n * 8 + e] + (p.y_bias ? p.y_bias[gc + n * 8 + e] : 0.f) : 0.f;
+      }
+    }
+#pragma unroll
+    for (int n = 0; n < 4; ++n) {
+      if (lc + n * 8 >= p.bs) continue;
+      float a[2], v[2];
+#pragma unroll
+      for (int e = 0; e < 2; ++e) {
+        const float la = -p.c * mg_sigmoid(acc[n][2 * half + e] + br[n][e]) * softplus_f(lam[n][e]);
+        a[e] = expf(la);
+        v[e] = sqrtf(-expm1f(2.f * la)) * mg_sigmoid(acc[n + 4][2 * half + e] + bi[n][e]) * (e ? u[n].y : u[n].x);
+      }
+      if (single) {
+#pragma unroll
+        for (int e = 0; e < 2; ++e) {
+          const float s = fmaf(a[e], S[n][e], v[e]);
+          st[n * 8 + e] = s;
+          mg_store<CT>(p.out, static_cast<size_t>(t) * p.ld_out + gc + n * 8 + e, s * gelu_tanh_f(y[n][e]));
+        }
+      } else {
+        float* o = p.ab + static_cast<size_t>(t) * 2 * p.C + gc + n * 8;
+        *reinterpret_cast<float2*>(o) = make_float2(a[0], a[1]);
+        *reinterpret_cast<float2*>(o + p.C) = make_float2(v[0], v[1]);
+      }
+    }
+  }
+}
+
 // requests that bring several rows, in order: one thread per (request, channel)
 template <typename CT>
 __global__ void __launch_bounds__(128) rglru_walk_kernel(RgLruParams p) {
@@ -428,7 +569,11 @@ int vb_rglru(void* d_out, int ld_out, float* d_state, float* d_ab, float* d_scra
                 d_slots, T, B, width, bs, c, n_tiles, tile_rows, d_tile_req, d_tile_row0, d_scratch};
   const bool f32 = out_dtype == 1;
   const dim3 grid(blocks * ((bs + RG_CH - 1) / RG_CH), (T + RG_R - 1) / RG_R);
-  if (w_dtype == 1) {
+  if (w_dtype == 0 && bs % 16 == 0 && ld_u % 4 == 0 && reinterpret_cast<uintptr_t>(d_u) % 16 == 0 && reinterpret_cast<uintptr_t>(d_w) % 16 == 0) {
+    const dim3 mgrid(blocks * ((bs + RM_CH - 1) / RM_CH), (T + RM_R - 1) / RM_R);
+    if (f32) VB_LAUNCH_PDL(rglru_gates_mma_kernel<float>, mgrid, 128, 0, stream, p);
+    else VB_LAUNCH_PDL(rglru_gates_mma_kernel<bf16>, mgrid, 128, 0, stream, p);
+  } else if (w_dtype == 1) {
     if (f32) VB_LAUNCH_PDL((rglru_gates_kernel<float, float>), grid, 256, 0, stream, p);
     else VB_LAUNCH_PDL((rglru_gates_kernel<float, bf16>), grid, 256, 0, stream, p);
   } else {

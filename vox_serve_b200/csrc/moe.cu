@@ -203,18 +203,17 @@ __global__ void __launch_bounds__(256) moe_route_sigmoid_kernel(int32_t* __restr
   if (lane < top) wts[t * top + lane] = normalize ? my_val / (denom + 1e-20f) : my_val;
 }
 
-// one warp per token
+// one CTA per token
 template <typename XT>
 __global__ void __launch_bounds__(128) moe_route_table_kernel(int32_t* __restrict__ idx, float* __restrict__ wts,
                                                               float* __restrict__ shared_gate, const int32_t* __restrict__ ids,
                                                               const int32_t* __restrict__ table, const XT* __restrict__ h,
-                                                              const float* __restrict__ wsg, int T, int W, int vocab, int E,
-                                                              int top) {
+                                                              const float* __restrict__ wsg, int W, int vocab, int E, int top) {
+  __shared__ float red[4];
   pdl_sync();
-  const int t = blockIdx.x * 4 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
-  if (t >= T) return;
+  const int t = blockIdx.x;
   const int32_t* row = table + static_cast<size_t>(min(max(ids[t], 0), vocab - 1)) * top;
-  for (int c = lane; c < top; c += 32) {
+  for (int c = threadIdx.x; c < top; c += 128) {
     idx[static_cast<size_t>(t) * top + c] = min(max(row[c], 0), E - 1);
     wts[static_cast<size_t>(t) * top + c] = 1.f / top;
   }
@@ -222,7 +221,7 @@ __global__ void __launch_bounds__(128) moe_route_table_kernel(int32_t* __restric
   const XT* x = h + static_cast<size_t>(t) * W;
   float s = 0.f;
   if ((W & 7) == 0) {
-    for (int i = lane * 8; i < W; i += 256) {
+    for (int i = threadIdx.x * 8; i < W; i += 1024) {
       const float4 a = *reinterpret_cast<const float4*>(wsg + i), b = *reinterpret_cast<const float4*>(wsg + i + 4);
       float v[8];
       if constexpr (sizeof(XT) == 4) {
@@ -237,13 +236,15 @@ __global__ void __launch_bounds__(128) moe_route_table_kernel(int32_t* __restric
       s = fmaf(v[4], b.x, s); s = fmaf(v[5], b.y, s); s = fmaf(v[6], b.z, s); s = fmaf(v[7], b.w, s);
     }
   } else {
-    for (int i = lane; i < W; i += 32) {
+    for (int i = threadIdx.x; i < W; i += 128) {
       if constexpr (sizeof(XT) == 4) s = fmaf(x[i], wsg[i], s);
       else s = fmaf(__bfloat162float(x[i]), wsg[i], s);
     }
   }
   s = warp_sum(s);
-  if (lane == 0) shared_gate[t] = 1.f / (1.f + expf(-s));
+  if ((threadIdx.x & 31) == 0) red[threadIdx.x >> 5] = s;
+  __syncthreads();
+  if (threadIdx.x == 0) shared_gate[t] = 1.f / (1.f + expf(-(red[0] + red[1] + red[2] + red[3])));
 }
 
 // single CTA: E <= 1024 experts, any number of pairs
@@ -300,6 +301,31 @@ __global__ void moe_combine_kernel(float* __restrict__ y, const float* __restric
   pdl_sync();
   const size_t t = blockIdx.x;
   const float ss = shared_scale ? shared_scale[t] : 1.f;
+  if ((W & 3) == 0 && top <= 8) {       // 16-byte pieces, every choice's load in flight
+    float w[8];
+    const float* src[8];
+#pragma unroll
+    for (int c = 0; c < 8; ++c) {
+      w[c] = c < top ? wts[t * top + c] : 0.f;
+      src[c] = c < top ? expert_out + static_cast<size_t>(pair_row[t * top + c]) * W : nullptr;
+    }
+    for (int i = threadIdx.x * 4; i < W; i += blockDim.x * 4) {
+      float4 v[8], s = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll
+      for (int c = 0; c < 8; ++c)
+        if (c < top) v[c] = *reinterpret_cast<const float4*>(src[c] + i);
+      if (shared_out) s = *reinterpret_cast<const float4*>(shared_out + t * W + i);
+      float4 a = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll
+      for (int c = 0; c < 8; ++c)
+        if (c < top) {
+          a.x = fmaf(w[c], v[c].x, a.x); a.y = fmaf(w[c], v[c].y, a.y); a.z = fmaf(w[c], v[c].z, a.z); a.w = fmaf(w[c], v[c].w, a.w);
+        }
+      if (shared_out) { a.x = fmaf(ss, s.x, a.x); a.y = fmaf(ss, s.y, a.y); a.z = fmaf(ss, s.z, a.z); a.w = fmaf(ss, s.w, a.w); }
+      *reinterpret_cast<float4*>(y + t * W + i) = a;
+    }
+    return;
+  }
   for (int i = threadIdx.x; i < W; i += blockDim.x) {
     float a = 0.f;
     for (int c = 0; c < top; ++c)
@@ -422,8 +448,8 @@ int vb_moe_route_table(int32_t* d_idx, float* d_wts, float* d_shared_gate, const
   VB_CHECK_ARG(experts >= 1 && experts <= 1024 && top >= 1 && top <= 32 && top <= experts,
                "vb_moe_route_table: experts %d (<= 1024), top %d (<= 32, <= experts)", experts, top);
   if (T <= 0) return 0;
-  if (h_dtype == 1) VB_LAUNCH_PDL(moe_route_table_kernel<float>, (T + 3) / 4, 128, 0, stream, d_idx, d_wts, d_shared_gate, d_ids, d_table, static_cast<const float*>(d_h), d_shared_gate_w, T, width, vocab, experts, top);
-  else VB_LAUNCH_PDL(moe_route_table_kernel<__nv_bfloat16>, (T + 3) / 4, 128, 0, stream, d_idx, d_wts, d_shared_gate, d_ids, d_table, static_cast<const __nv_bfloat16*>(d_h), d_shared_gate_w, T, width, vocab, experts, top);
+  if (h_dtype == 1) VB_LAUNCH_PDL(moe_route_table_kernel<float>, T, 128, 0, stream, d_idx, d_wts, d_shared_gate, d_ids, d_table, static_cast<const float*>(d_h), d_shared_gate_w, width, vocab, experts, top);
+  else VB_LAUNCH_PDL(moe_route_table_kernel<__nv_bfloat16>, T, 128, 0, stream, d_idx, d_wts, d_shared_gate, d_ids, d_table, static_cast<const __nv_bfloat16*>(d_h), d_shared_gate_w, width, vocab, experts, top);
   return 0;
 }
 

@@ -24,6 +24,13 @@ template <> __device__ __forceinline__ float sd_to_f<float>(float v) { return v;
 template <> __device__ __forceinline__ float sd_to_f<__nv_bfloat16>(__nv_bfloat16 v) { return __bfloat162float(v); }
 __device__ __forceinline__ float sd_softplus(float v) { return fmaxf(v, 0.f) + log1pf(expf(-fabsf(v))); }
 __device__ __forceinline__ float sd_silu(float z) { return z / (1.f + expf(-z)); }
+// two fp32 values as bf16 terms: the rounded values, and (lo) what the rounding left
+__device__ __forceinline__ uint32_t sd_split(float a, float b, uint32_t& lo) {
+  const __nv_bfloat16 ha = __float2bfloat16_rn(a), hb = __float2bfloat16_rn(b);
+  lo = pack_bf16(a - __bfloat162float(ha), b - __bfloat162float(hb));
+  return pack_bf16(__bfloat162float(ha), __bfloat162float(hb));
+}
+
 
 struct SsdParams {
   const void* xbc;        // [T][ld]: x [H * V] | B [G * N] | C [G * N]
@@ -45,7 +52,8 @@ struct SsdParams {
   // tiled form
   const int32_t* tile_req;
   const int32_t* tile_row0;
-  float* scratch;         // [tiles][H][N][V]: local end states, then the states before the tiles
+  float* scratch;         // [tiles][H][N][V]: local end states; fp32 form: then the states before the tiles
+  __nv_bfloat16* before;  // tensor-core form: the states before the tiles as [tiles][H][2][N][V], rounded and the remainder
   float* tile_decay;      // [tiles][H]: the tile's whole decay
 };
 
@@ -226,7 +234,7 @@ __global__ void __launch_bounds__(256) ssd_tile_state_kernel(SsdParams p) {
   }
 }
 
-// per request: scratch[tile] <- the state before the tile, the slot <- the state after the last one
+// per request: scratch[tile] (or before[tile]) <- the state before the tile, the slot <- the state after the last one
 __global__ void __launch_bounds__(256) ssd_tile_scan_kernel(SsdParams p) {
   pdl_sync();
   const int b = blockIdx.x, h = blockIdx.y;
@@ -243,6 +251,37 @@ __global__ void __launch_bounds__(256) ssd_tile_scan_kernel(SsdParams p) {
   float* S = p.state + (static_cast<size_t>(p.slots[b]) * p.H + h) * per;
   const float* dec = p.tile_decay + static_cast<size_t>(first) * p.H + h;
   float* sc = p.scratch + (static_cast<size_t>(first) * p.H + h) * per;
+  if (per % 4 == 0 && ((reinterpret_cast<uintptr_t>(S) | reinterpret_cast<uintptr_t>(sc)) & 15) == 0) {
+    // four neighbouring values per thread in 16-byte pieces (the grid covers them once)
+    const size_t i = (static_cast<size_t>(blockIdx.z) * blockDim.x + threadIdx.x) * 4, step = static_cast<size_t>(p.H) * per;
+    if (i >= per) return;
+    float4 s = fresh ? make_float4(0.f, 0.f, 0.f, 0.f) : *reinterpret_cast<const float4*>(S + i);
+    for (int c0 = 0; c0 < n_tiles; c0 += 8) {
+      float4 uv[8];
+#pragma unroll
+      for (int j = 0; j < 8; ++j)
+        if (c0 + j < n_tiles) uv[j] = *reinterpret_cast<const float4*>(sc + (c0 + j) * step + i);
+#pragma unroll
+      for (int j = 0; j < 8; ++j) {
+        if (c0 + j < n_tiles) {
+          if (p.before) {
+            __nv_bfloat16* o = p.before + (static_cast<size_t>(first + c0 + j) * p.H + h) * 2 * per + i;
+            uint2 hi, lo;
+            hi.x = sd_split(s.x, s.y, lo.x);
+            hi.y = sd_split(s.z, s.w, lo.y);
+            *reinterpret_cast<uint2*>(o) = hi;
+            *reinterpret_cast<uint2*>(o + per) = lo;
+          } else {
+            *reinterpret_cast<float4*>(sc + (c0 + j) * step + i) = s;
+          }
+          const float d = dec[static_cast<size_t>(c0 + j) * p.H];
+          s.x = fmaf(d, s.x, uv[j].x); s.y = fmaf(d, s.y, uv[j].y); s.z = fmaf(d, s.z, uv[j].z); s.w = fmaf(d, s.w, uv[j].w);
+        }
+      }
+    }
+    *reinterpret_cast<float4*>(S + i) = s;
+    return;
+  }
   for (size_t i = blockIdx.z * blockDim.x + threadIdx.x; i < per; i += static_cast<size_t>(gridDim.z) * blockDim.x) {
     float s = fresh ? 0.f : S[i];
     for (int c0 = 0; c0 < n_tiles; c0 += 8) {          // eight independent loads in flight, then the serial update
@@ -380,6 +419,234 @@ __global__ void __launch_bounds__(256) ssd_tile_out_kernel(SsdParams p) {
   }
 }
 
+// ------------------------------------------------------------------------------------------------------------------
+// The tiles on the tensor cores (bf16 rows, N and V multiples of 16): CTA = (64-row tile, one or several heads of a group, up
+// to 64 value dims), mma.sync m16n8k16 with fp32 accumulators.  B, C and x are bf16 as they stand; an fp32 operand (the
+// decayed weights, the weighted x, the state) enters as two bf16 terms, its rounding and the remainder's, so that a product keeps
+// 16 bits of its mantissa.
+// ------------------------------------------------------------------------------------------------------------------
+// rows [0, L) x n columns of bf16 (16-byte pieces) into smem [64][ld], zeros below
+__device__ __forceinline__ void sd_stage(__nv_bfloat16* __restrict__ dst, int ld, const __nv_bfloat16* __restrict__ src, int ld_src, int n,
+                                         int L) {
+  const int v = n / 8;
+  for (int i = threadIdx.x; i < SD_ROWS * v; i += 128) {
+    const int r = i / v, c = (i - r * v) * 8;
+    uint4 q = make_uint4(0u, 0u, 0u, 0u);
+    if (r < L) q = *reinterpret_cast<const uint4*>(src + static_cast<size_t>(r) * ld_src + c);
+    *reinterpret_cast<uint4*>(dst + r * ld + c) = q;
+  }
+}
+
+__global__ void __launch_bounds__(128) ssd_tile_state_mma_kernel(SsdParams p, int hb) {
+  extern __shared__ __align__(16) uint8_t sd_raw[];
+  __shared__ float dts[SD_ROWS];
+  __shared__ double cum[SD_ROWS];
+  pdl_sync();
+  const int tile = blockIdx.x, h0 = blockIdx.y * hb, e0 = blockIdx.z * p.dvb, g = h0 / (p.H / p.G);
+  const int row0 = p.tile_row0[tile], L = min(SD_ROWS, p.qo_indptr[p.tile_req[tile] + 1] - row0);
+  const int N = p.N, V = p.V, DV = min(p.dvb, V - e0), ldb = N + 8, ldx = p.dvb + 8;
+  __nv_bfloat16* Bs = reinterpret_cast<__nv_bfloat16*>(sd_raw);       // [64][N + 8]
+  __nv_bfloat16* Xh = Bs + SD_ROWS * ldb;                             // [64][dvb + 8] the weighted x, and its remainder
+  __nv_bfloat16* Xl = Xh + SD_ROWS * ldx;
+  const __nv_bfloat16* xbc = static_cast<const __nv_bfloat16*>(p.xbc) + static_cast<size_t>(row0) * p.ld;
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, vb = DV / 8;
+  sd_stage(Bs, ldb, xbc + p.H * V + g * N, p.ld, N, L);
+  for (int h = h0; h < h0 + hb; ++h) {
+    __syncthreads();                      // (the last head's x is consumed)
+    ssd_tile_decays(p, h, row0, L, dts, cum);
+    const double last = cum[L - 1];
+    if (tid == 0 && blockIdx.z == 0) p.tile_decay[static_cast<size_t>(tile) * p.H + h] = static_cast<float>(exp(last));
+    for (int i = tid; i < SD_ROWS * vb; i += 128) {
+      const int r = i / vb, c = (i - r * vb) * 8;
+      uint4 hi = make_uint4(0u, 0u, 0u, 0u), lo = hi;
+      if (r < L) {
+        const float w = expf(static_cast<float>(last - cum[r])) * dts[r];
+        const uint4 q = *reinterpret_cast<const uint4*>(xbc + static_cast<size_t>(r) * p.ld + h * V + e0 + c);
+        hi.x = sd_split(w * bf16_lo(q.x), w * bf16_hi(q.x), lo.x);
+        hi.y = sd_split(w * bf16_lo(q.y), w * bf16_hi(q.y), lo.y);
+        hi.z = sd_split(w * bf16_lo(q.z), w * bf16_hi(q.z), lo.z);
+        hi.w = sd_split(w * bf16_lo(q.w), w * bf16_hi(q.w), lo.w);
+      }
+      *reinterpret_cast<uint4*>(Xh + r * ldx + c) = hi;
+      *reinterpret_cast<uint4*>(Xl + r * ldx + c) = lo;
+    }
+    __syncthreads();
+    float* U = p.scratch + (static_cast<size_t>(tile) * p.H + h) * N * V + e0;
+    for (int m0 = warp * 16; m0 < N; m0 += 64) {
+      float acc[8][4];
+#pragma unroll
+      for (int n = 0; n < 8; ++n) acc[n][0] = acc[n][1] = acc[n][2] = acc[n][3] = 0.f;
+#pragma unroll
+      for (int kb = 0; kb < SD_ROWS / 16; ++kb) {
+        uint32_t af[4];                   // B^T: the stored rows are k, transposed on the way into registers
+        ldmatrix_x4_trans(af, smem_u32(Bs + (kb * 16 + (lane >> 4) * 8 + (lane & 7)) * ldb + m0 + ((lane >> 3) & 1) * 8));
+#pragma unroll
+        for (int np = 0; np < 4; ++np) {
+          if (np * 16 < DV) {
+            const int off = (kb * 16 + ((lane >> 3) & 1) * 8 + (lane & 7)) * ldx + np * 16 + (lane >> 4) * 8;
+            uint32_t bh[4], bl[4];
+            ldmatrix_x4_trans(bh, smem_u32(Xh + off));
+            ldmatrix_x4_trans(bl, smem_u32(Xl + off));
+            mma_bf16_16816(acc[2 * np], af, bh[0], bh[1]);
+            mma_bf16_16816(acc[2 * np], af, bl[0], bl[1]);
+            mma_bf16_16816(acc[2 * np + 1], af, bh[2], bh[3]);
+            mma_bf16_16816(acc[2 * np + 1], af, bl[2], bl[3]);
+          }
+        }
+      }
+#pragma unroll
+      for (int n = 0; n < 8; ++n) {
+        const int c = n * 8 + (lane & 3) * 2;
+        if (c < DV) {
+          float* u = U + static_cast<size_t>(m0 + (lane >> 2)) * V + c;
+          *reinterpret_cast<float2*>(u) = make_float2(acc[n][0], acc[n][1]);
+          *reinterpret_cast<float2*>(u + static_cast<size_t>(8) * V) = make_float2(acc[n][2], acc[n][3]);
+        }
+      }
+    }
+  }
+}
+
+// 8 warps: warp w owns the 16 rows of w / 2 and one half of the value dims
+__global__ void __launch_bounds__(256) ssd_tile_out_mma_kernel(SsdParams p) {
+  extern __shared__ __align__(16) uint8_t sd_raw[];
+  __shared__ float dts[SD_ROWS], cumf[SD_ROWS];
+  __shared__ double cum[SD_ROWS];
+  const int tile = blockIdx.x, h = blockIdx.y, e0 = blockIdx.z * p.dvb, g = h / (p.H / p.G);
+  const int row0 = p.tile_row0[tile], L = min(SD_ROWS, p.qo_indptr[p.tile_req[tile] + 1] - row0);
+  const int N = p.N, V = p.V, DV = min(p.dvb, V - e0), ldb = N + 8, ldx = p.dvb + 8, nkb = N / 16;
+  __nv_bfloat16* Cs = reinterpret_cast<__nv_bfloat16*>(sd_raw);       // [64][N + 8]
+  __nv_bfloat16* Bs = Cs + SD_ROWS * ldb;                             // [64][N + 8]
+  __nv_bfloat16* Xs = Bs + SD_ROWS * ldb;                             // [64][dvb + 8]
+  __nv_bfloat16* Sh = Xs + SD_ROWS * ldx;                             // [N][dvb + 8] the state before the tile, and its remainder
+  __nv_bfloat16* Sl = Sh + N * ldx;
+  const __nv_bfloat16* xbc = static_cast<const __nv_bfloat16*>(p.xbc) + static_cast<size_t>(row0) * p.ld;
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  // every copy is in flight before anything is waited for: B and C first (the scores need them), then x and the state
+  auto copy = [&](__nv_bfloat16* dst, int ld, const __nv_bfloat16* src, int ld_src, int n, int rows, int valid) {
+    const int v = n / 8;
+    for (int i = tid; i < rows * v; i += 256) {
+      const int r = i / v, c = (i - r * v) * 8;
+      asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(smem_u32(dst + r * ld + c)),
+                   "l"(src + static_cast<size_t>(r < valid ? r : 0) * ld_src + c), "r"(r < valid ? 16u : 0u) : "memory");
+    }
+  };
+  pdl_sync();
+  copy(Bs, ldb, xbc + p.H * V + g * N, p.ld, N, SD_ROWS, L);
+  copy(Cs, ldb, xbc + p.H * V + p.G * N + g * N, p.ld, N, SD_ROWS, L);
+  asm volatile("cp.async.commit_group;" ::: "memory");
+  const __nv_bfloat16* Sb = p.before + (static_cast<size_t>(tile) * p.H + h) * 2 * N * V + e0;
+  copy(Xs, ldx, xbc + h * V + e0, p.ld, DV, SD_ROWS, L);
+  copy(Sh, ldx, Sb, V, DV, N, N);
+  copy(Sl, ldx, Sb + static_cast<size_t>(N) * V, V, DV, N, N);
+  asm volatile("cp.async.commit_group;" ::: "memory");
+  ssd_tile_decays(p, h, row0, L, dts, cum);
+  if (tid < SD_ROWS) cumf[tid] = static_cast<float>(cum[tid]);
+  asm volatile("cp.async.wait_group 1;" ::: "memory");
+  __syncthreads();
+  // scores of the warp's 16 rows with the rows up to its last one
+  const int rb = warp >> 1, v0 = (warp & 1) * 32;
+  const __nv_bfloat16* Crow = Cs + (rb * 16 + (lane & 15)) * ldb + (lane >> 4) * 8;
+  float sc[8][4];
+#pragma unroll
+  for (int n = 0; n < 8; ++n) sc[n][0] = sc[n][1] = sc[n][2] = sc[n][3] = 0.f;
+  for (int kb = 0; kb < nkb; ++kb) {
+    uint32_t af[4];
+    ldmatrix_x4(af, smem_u32(Crow + kb * 16));
+#pragma unroll
+    for (int np = 0; np < 4; ++np) {
+      if (np <= rb) {
+        uint32_t bf[4];
+        ldmatrix_x4(bf, smem_u32(Bs + (np * 16 + (lane >> 4) * 8 + (lane & 7)) * ldb + kb * 16 + ((lane >> 3) & 1) * 8));
+        mma_bf16_16816(sc[2 * np], af, bf[0], bf[1]);
+        mma_bf16_16816(sc[2 * np + 1], af, bf[2], bf[3]);
+      }
+    }
+  }
+  asm volatile("cp.async.wait_group 0;" ::: "memory");
+  __syncthreads();
+  if (v0 >= DV) return;
+  const int rA = rb * 16 + (lane >> 2), rB = rA + 8;
+  float o[4][4];
+#pragma unroll
+  for (int n = 0; n < 4; ++n) o[n][0] = o[n][1] = o[n][2] = o[n][3] = 0.f;
+  // what the state before the tile contributes
+  for (int kb = 0; kb < nkb; ++kb) {
+    uint32_t af[4];
+    ldmatrix_x4(af, smem_u32(Crow + kb * 16));
+#pragma unroll
+    for (int np = 0; np < 2; ++np) {
+      if (v0 + np * 16 < DV) {
+        const int off = (kb * 16 + ((lane >> 3) & 1) * 8 + (lane & 7)) * ldx + v0 + np * 16 + (lane >> 4) * 8;
+        uint32_t bh[4], bl[4];
+        ldmatrix_x4_trans(bh, smem_u32(Sh + off));
+        ldmatrix_x4_trans(bl, smem_u32(Sl + off));
+        mma_bf16_16816(o[2 * np], af, bh[0], bh[1]);
+        mma_bf16_16816(o[2 * np + 1], af, bh[2], bh[3]);
+        mma_bf16_16816(o[2 * np], af, bl[0], bl[1]);
+        mma_bf16_16816(o[2 * np + 1], af, bl[2], bl[3]);
+      }
+    }
+  }
+  const float cA = cumf[rA], cB = cumf[rB], dA = expf(cA), dB = expf(cB);
+#pragma unroll
+  for (int n = 0; n < 4; ++n) { o[n][0] *= dA; o[n][1] *= dA; o[n][2] *= dB; o[n][3] *= dB; }
+  // the tile's own rows
+#pragma unroll
+  for (int kb = 0; kb < SD_ROWS / 16; ++kb) {
+    if (kb <= rb) {
+      float m[2][4];
+#pragma unroll
+      for (int u = 0; u < 2; ++u)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+          const int j = kb * 16 + u * 8 + (lane & 3) * 2 + (e & 1);
+          const bool ok = j <= (e < 2 ? rA : rB);
+          m[u][e] = ok ? sc[2 * kb + u][e] * expf((e < 2 ? cA : cB) - cumf[j]) * dts[j] : 0.f;
+        }
+      uint32_t ah[4], al[4];
+      ah[0] = sd_split(m[0][0], m[0][1], al[0]);
+      ah[1] = sd_split(m[0][2], m[0][3], al[1]);
+      ah[2] = sd_split(m[1][0], m[1][1], al[2]);
+      ah[3] = sd_split(m[1][2], m[1][3], al[3]);
+#pragma unroll
+      for (int np = 0; np < 2; ++np) {
+        if (v0 + np * 16 < DV) {
+          uint32_t xf[4];
+          ldmatrix_x4_trans(xf, smem_u32(Xs + (kb * 16 + ((lane >> 3) & 1) * 8 + (lane & 7)) * ldx + v0 + np * 16 + (lane >> 4) * 8));
+          mma_bf16_16816(o[2 * np], ah, xf[0], xf[1]);
+          mma_bf16_16816(o[2 * np + 1], ah, xf[2], xf[3]);
+          mma_bf16_16816(o[2 * np], al, xf[0], xf[1]);
+          mma_bf16_16816(o[2 * np + 1], al, xf[2], xf[3]);
+        }
+      }
+    }
+  }
+  const float D = p.D[h];
+#pragma unroll
+  for (int half = 0; half < 2; ++half) {
+    const int r = half ? rB : rA;
+    if (r >= L) continue;
+    const size_t t = row0 + r;
+    const float* z = p.z + t * p.ld_z + h * V + e0;
+    float* out = p.out + t * p.H * V + h * V + e0;
+#pragma unroll
+    for (int n = 0; n < 4; ++n) {
+      const int c = v0 + n * 8 + (lane & 3) * 2;
+      if (c < DV) {
+        const uint32_t x = *reinterpret_cast<const uint32_t*>(Xs + r * ldx + c);
+        const float y0 = fmaf(D, bf16_lo(x), o[n][2 * half]), y1 = fmaf(D, bf16_hi(x), o[n][2 * half + 1]);
+        *reinterpret_cast<float2*>(out + c) = make_float2(y0 * sd_silu(z[c]), y1 * sd_silu(z[c + 1]));
+      }
+    }
+  }
+}
+
+static size_t ssd_mma_smem1(int N, int dvb) { return (static_cast<size_t>(SD_ROWS) * (N + 8) + 2ull * SD_ROWS * (dvb + 8)) * 2; }
+static size_t ssd_mma_smem3(int N, int dvb) {
+  return (2ull * SD_ROWS * (N + 8) + static_cast<size_t>(SD_ROWS) * (dvb + 8) + 2ull * N * (dvb + 8)) * 2;
+}
+
 // one CTA per (row, neighbourhood of n channels)
 template <typename OT>
 __global__ void __launch_bounds__(256) group_rmsnorm_kernel(OT* __restrict__ out, const float* __restrict__ x,
@@ -403,6 +670,40 @@ __global__ void __launch_bounds__(256) group_rmsnorm_kernel(OT* __restrict__ out
     if constexpr (sizeof(OT) == 4) o[i] = v;
     else o[i] = __float2bfloat16_rn(v);
   }
+}
+
+// one warp per (row, neighbourhood) in 16-byte pieces: n a multiple of 4, at most 1024
+template <typename OT>
+__global__ void __launch_bounds__(256) group_rmsnorm_warp_kernel(OT* __restrict__ out, const float* __restrict__ x,
+                                                                 const float* __restrict__ w, int groups, int n, long long rows,
+                                                                 float eps) {
+  pdl_sync();
+  const long long i = static_cast<long long>(blockIdx.x) * 8 + (threadIdx.x >> 5);
+  if (i >= rows) return;
+  const int lane = threadIdx.x & 31, n4 = n >> 2;
+  const float4* src = reinterpret_cast<const float4*>(x + i * n);
+  const float4* wt = reinterpret_cast<const float4*>(w + (i % groups) * n);
+  float4 v[8];
+  float q = 0.f;
+#pragma unroll
+  for (int j = 0; j < 8; ++j)
+    if (lane + 32 * j < n4) v[j] = src[lane + 32 * j];
+#pragma unroll
+  for (int j = 0; j < 8; ++j)
+    if (lane + 32 * j < n4) {
+      q = fmaf(v[j].x, v[j].x, q); q = fmaf(v[j].y, v[j].y, q); q = fmaf(v[j].z, v[j].z, q); q = fmaf(v[j].w, v[j].w, q);
+    }
+  const float rs = 1.f / sqrtf(warp_sum(q) / n + eps);
+  OT* o = out + i * n;
+#pragma unroll
+  for (int j = 0; j < 8; ++j)
+    if (lane + 32 * j < n4) {
+      const int c = lane + 32 * j;
+      const float4 ww = wt[c];
+      const float a = v[j].x * rs * ww.x, b = v[j].y * rs * ww.y, d = v[j].z * rs * ww.z, e = v[j].w * rs * ww.w;
+      if constexpr (sizeof(OT) == 4) reinterpret_cast<float4*>(o)[c] = make_float4(a, b, d, e);
+      else reinterpret_cast<uint2*>(o)[c] = make_uint2(pack_bf16(a, b), pack_bf16(d, e));
+    }
 }
 
 static int ssd_dvb(int V) {
@@ -457,7 +758,7 @@ int vb_ssd_tile_rows(int V, int N) {
 }
 
 long long vb_ssd_scratch_floats(int n_tiles, int H, int V, int N) {
-  return static_cast<long long>(n_tiles) * H * (static_cast<long long>(N) * V + 1);
+  return static_cast<long long>(n_tiles) * H * (2ll * N * V + 1);
 }
 
 int vb_ssd_tiled(float* d_out, float* d_state, float* d_scratch, const void* d_xbc, int ld, const float* d_dt, int ld_dt,
@@ -474,7 +775,7 @@ int vb_ssd_tiled(float* d_out, float* d_state, float* d_scratch, const void* d_x
   p.state = d_state; p.out = d_out; p.qo_indptr = d_qo_indptr; p.pos = d_pos; p.slots = d_slots;
   p.H = H; p.V = V; p.N = N; p.G = G; p.dvb = ssd_dvb(V); p.min_rows = 2; p.max_rows = 1 << 30;
   p.tile_req = d_tile_req; p.tile_row0 = d_tile_row0; p.scratch = d_scratch;
-  p.tile_decay = d_scratch + static_cast<size_t>(n_tiles) * H * N * V;
+  p.tile_decay = d_scratch + 2 * static_cast<size_t>(n_tiles) * H * N * V;
   const int zb = (V + p.dvb - 1) / p.dvb;
   const size_t per = static_cast<size_t>(N) * V;
   const size_t smem1 = static_cast<size_t>(SD_ROWS) * (N + 1 + p.dvb + 1) * sizeof(float), smem3 = ssd_out_smem(N, p.dvb);
@@ -485,6 +786,19 @@ int vb_ssd_tiled(float* d_out, float* d_state, float* d_scratch, const void* d_x
     VB_LAUNCH_PDL(ssd_tile_state_kernel<float>, grid, 256, smem1, stream, p);
     VB_LAUNCH_PDL(ssd_tile_scan_kernel, scan_grid, 256, 0, stream, p);
     VB_LAUNCH_PDL(ssd_tile_out_kernel<float>, grid, 256, smem3, stream, p);
+  } else if (N % 16 == 0 && V % 16 == 0 && ld % 8 == 0 && ssd_mma_smem3(N, p.dvb) <= static_cast<size_t>(VB_MAX_DYN_SMEM) - 2048 &&
+             ((reinterpret_cast<uintptr_t>(d_xbc) | reinterpret_cast<uintptr_t>(d_scratch) | reinterpret_cast<uintptr_t>(d_state)) & 15) == 0 &&
+             reinterpret_cast<uintptr_t>(d_out) % 8 == 0) {
+    // several heads of a group per CTA where that leaves two CTAs per SM
+    int hb = 1;
+    while (hb < 4 && (H / G) % (2 * hb) == 0 && n_tiles * (H / (2 * hb)) * zb >= 2 * 148) hb *= 2;
+    p.before = reinterpret_cast<bf16*>(d_scratch + static_cast<size_t>(n_tiles) * H * N * V);
+    const dim3 mgrid(n_tiles, H / hb, zb);
+    VB_CHECK_CUDA(cudaFuncSetAttribute(ssd_tile_state_mma_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, VB_MAX_DYN_SMEM - 2048));
+    VB_CHECK_CUDA(cudaFuncSetAttribute(ssd_tile_out_mma_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, VB_MAX_DYN_SMEM - 2048));
+    VB_LAUNCH_PDL(ssd_tile_state_mma_kernel, mgrid, 128, ssd_mma_smem1(N, p.dvb), stream, p, hb);
+    VB_LAUNCH_PDL(ssd_tile_scan_kernel, scan_grid, 256, 0, stream, p);
+    VB_LAUNCH_PDL(ssd_tile_out_mma_kernel, grid, 256, ssd_mma_smem3(N, p.dvb), stream, p);
   } else {
     VB_CHECK_CUDA(cudaFuncSetAttribute(ssd_tile_state_kernel<bf16>, cudaFuncAttributeMaxDynamicSharedMemorySize, VB_MAX_DYN_SMEM - 2048));
     VB_CHECK_CUDA(cudaFuncSetAttribute(ssd_tile_out_kernel<bf16>, cudaFuncAttributeMaxDynamicSharedMemorySize, VB_MAX_DYN_SMEM - 2048));
@@ -500,6 +814,14 @@ int vb_group_rmsnorm(void* d_out, const float* d_x, const float* d_w, int T, int
   VB_CHECK_ARG(d_out && d_x && d_w && C > 0 && groups > 0 && C % groups == 0, "vb_group_rmsnorm: %d channels in %d groups", C, groups);
   if (T <= 0) return 0;
   const dim3 grid(T, groups);
+  const int n = C / groups;
+  if (n % 4 == 0 && n <= 1024 && ((reinterpret_cast<uintptr_t>(d_x) | reinterpret_cast<uintptr_t>(d_w) | reinterpret_cast<uintptr_t>(d_out)) & 15) == 0) {
+    const long long rows = static_cast<long long>(T) * groups;
+    const unsigned blocks = static_cast<unsigned>((rows + 7) / 8);
+    if (out_dtype == 1) VB_LAUNCH_PDL(group_rmsnorm_warp_kernel<float>, blocks, 256, 0, stream, static_cast<float*>(d_out), d_x, d_w, groups, n, rows, eps);
+    else VB_LAUNCH_PDL(group_rmsnorm_warp_kernel<bf16>, blocks, 256, 0, stream, static_cast<bf16*>(d_out), d_x, d_w, groups, n, rows, eps);
+    return 0;
+  }
   if (out_dtype == 1) VB_LAUNCH_PDL(group_rmsnorm_kernel<float>, grid, 256, 0, stream, static_cast<float*>(d_out), d_x, d_w, C, C / groups, eps);
   else VB_LAUNCH_PDL(group_rmsnorm_kernel<bf16>, grid, 256, 0, stream, static_cast<bf16*>(d_out), d_x, d_w, C, C / groups, eps);
   return 0;
