@@ -631,11 +631,11 @@ int vb_mingru_tiled(void* d_out, float* d_state, float* d_scratch, const float* 
 int vb_mingru_scratch_floats(int n_tiles, int tile_rows, int width);
 /* Real-gated linear recurrent unit over fp32 state slots [slots][width]: r = sigmoid(R_b u + br), i = sigmoid(I_b u + bi) in
  * `blocks` equal parts of the channels (d_w [blocks][2 * bs][bs]: R_b above I_b, bf16 or fp32; d_bias [blocks][2 * bs]),
- * log a = -c r softplus(d_lam), S_t = a S_(t-1) + sqrt(1 - a^2) i u, d_out = S * gelu_tanh(d_y + d_y_bias).  One launch serves
+ * log a = -d_rate r, S_t = a S_(t-1) + sqrt(1 - a^2) i u, d_out = S * gelu_tanh(d_y + d_y_bias).  One launch serves
  * requests that bring one row; multi_rows != 0: the others too, with d_ab fp32 [T][2][width], walked in order (n_tiles == 0)
  * or in the tiles and pieces of vb_mingru_tiled (d_scratch: vb_mingru_scratch_floats floats). */
 int vb_rglru(void* d_out, int ld_out, float* d_state, float* d_ab, float* d_scratch, const float* d_u, int ld_u, const void* d_w,
-             const float* d_bias, const float* d_lam, float c, const float* d_y, int ld_y, const float* d_y_bias,
+             const float* d_bias, const float* d_rate, const float* d_y, int ld_y, const float* d_y_bias,
              const int32_t* d_qo_indptr, const int32_t* d_row_req, const int32_t* d_pos, const int32_t* d_slots,
              const int32_t* d_tile_req, const int32_t* d_tile_row0, int n_tiles, int tile_rows, int T, int B, int width,
              int blocks, int multi_rows, int w_dtype, int out_dtype, void* stream);

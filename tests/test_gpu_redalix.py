@@ -317,15 +317,16 @@ TC = dict(width=128, vocab=160, a_heads=4, a_kv_heads=2, a_dim=32, a_vdim=48, a_
 
 
 @pytest.mark.gpu
-def test_bfloat16_tensor_core_sizes():
+@pytest.mark.parametrize("kw", [{}, dict(shared_ff=96), dict(shared_ff=0, top=1), dict(e_ff=96, top=1), dict(experts=20, top=1)])
+def test_bfloat16_tensor_core_sizes(kw):
     """sizes whose projections, attention, recurrence gates and state-space tiles run on the tensor-core kernels: a 600-token prompt
     whole (grouped experts, tiles) against portions (single rows among them), against the plain projection kernel with the recurrences
-    row by row, and against the oracle"""
-    cfg = O.make_config(layers=("mamba:moe", "pair:moe", "attn:moe", "pair:dense"), **TC)
+    row by row, and against the oracle; expert widths and counts that take the grouped and the stacked form and neither"""
+    cfg = O.make_config(layers=("mamba:moe", "pair:moe", "attn:moe", "pair:dense"), **{**TC, **kw})
     sd = O.make_weights(cfg, 21)
     toks = _tokens(600, cfg["vocab"], 6)
     ref = O.forward(cfg, sd, toks)
-    kw = dict(slots=2, pages=24, page_size=64, max_rows=1024)
+    kw = dict(slots=2, pages=24, page_size=64, max_rows=1024)          # (the worker's)
     cuts = [[("a", 130)], [("a", 1)], [("a", 300)], [("a", 2)], [("a", 167)]]
     w = _worker(cfg, sd, BF16, **kw)
     whole, parts = _replay(w, {"a": toks}, [[("a", 600)]])["a"], _replay(w, {"a": toks}, cuts)["a"]
@@ -512,7 +513,7 @@ def test_gated_linear_recurrence(dtype, tiled, C, blocks):
         S, _ = O.linear_recurrent_unit(u, O.gate_blocks(u, ra.double(), rb.double()), O.gate_blocks(u, ri.double(), ib.double()), lam.double())
         ref.append(S * O.gelu_tanh(y + yb.double()))
     w = torch.cat([ra, ri], 1).to(wt).to(DEV).contiguous()
-    bias = torch.cat([rb, ib], 1).to(DEV).contiguous()
+    bias, rate = torch.cat([rb, ib], 1).to(DEV).contiguous(), (8.0 * O.softplus(lam.double())).to(F32).to(DEV)
     for cuts in CUTS:
         state = torch.full((7, C), float("nan"), dtype=F32, device=DEV)
         outs = [[] for _ in lens]
@@ -523,7 +524,7 @@ def test_gated_linear_recurrence(dtype, tiled, C, blocks):
             wide = torch.zeros(T, 2 * C + 4, device=DEV)
             wide[:, :C], wide[:, C + 4:] = u, y
             out = torch.zeros(T, C, dtype=dtype, device=DEV)
-            ops.rglru(wide[:, :C], w, bias, lam.to(DEV), 8.0, wide[:, C + 4:], yb.to(DEV), state, out, torch.zeros(2 * T * C, device=DEV), qo,
+            ops.rglru(wide[:, :C], w, bias, rate, wide[:, C + 4:], yb.to(DEV), state, out, torch.zeros(2 * T * C, device=DEV), qo,
                       row_req, pos, slots, len(live), multi_rows=tiles is not None, tiles=(*tiles, 64) if (tiles and tiled) else None,
                       scratch=torch.zeros(ops.mingru_scratch_floats(tiles[2], 64, C) if tiles else 1, device=DEV))
             for i, (b, _, n) in enumerate(live):
@@ -544,12 +545,12 @@ def test_split_products_of_the_gates_keep_fp32_accuracy():
     T, C, blocks = 70, 256, 2
     u, y = torch.randn(T, C, generator=g).to(DEV) * 2, torch.randn(T, C, generator=g).to(DEV)
     w = (torch.randn(blocks, 2 * C // blocks, C // blocks, generator=g) * 0.15).to(BF16).to(DEV)
-    bias, lam = torch.randn(blocks, 2 * C // blocks, generator=g).to(DEV), torch.randn(C, generator=g).to(DEV) - 4
+    bias, rate = torch.randn(blocks, 2 * C // blocks, generator=g).to(DEV), 8.0 * O.softplus(torch.randn(C, generator=g) - 4).to(DEV)
     qo, row_req, pos = _step_tables([(0, T)])
     got = []
     for wt in (BF16, F32):
         ab = torch.zeros(2 * T * C, device=DEV)
-        ops.rglru(u, w.to(wt), bias, lam, 8.0, y, None, torch.zeros(1, C, device=DEV), torch.zeros(T, C, device=DEV), ab, qo, row_req, pos,
+        ops.rglru(u, w.to(wt), bias, rate, y, None, torch.zeros(1, C, device=DEV), torch.zeros(T, C, device=DEV), ab, qo, row_req, pos,
                   torch.zeros(1, dtype=I32, device=DEV), 1)
         got.append(ab)
     assert (got[0] - got[1]).abs().max().item() < 1e-4 and (got[0] - got[1]).pow(2).mean().sqrt().item() < 5e-6

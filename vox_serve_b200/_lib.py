@@ -162,7 +162,7 @@ SIGNATURES = {
     "vb_hyper_mix_norm": (c_int, [P, c_int, P, P, P, P, P, P, P, P, P, c_int, c_int, c_float, P, c_int, P, P, P, c_int, c_int, P]),
     "vb_short_conv": (c_int, [P, c_int, P, c_int, P, c_int, P, P, P, P, P, P, P, c_int, c_int, c_int, c_int, c_int, c_int, c_int,
                               P, P]),
-    "vb_rglru": (c_int, [P, c_int, P, P, P, P, c_int, P, P, P, c_float, P, c_int, P, P, P, P, P, P, P, c_int, c_int, c_int, c_int,
+    "vb_rglru": (c_int, [P, c_int, P, P, P, P, c_int, P, P, P, P, c_int, P, P, P, P, P, P, P, c_int, c_int, c_int, c_int,
                          c_int, c_int, c_int, c_int, c_int, P]),
     "vb_ssd": (c_int, [P, P, P, c_int, P, c_int, P, P, P, P, c_int, P, P, P, c_int, c_int, c_int, c_int, c_int, c_int, c_int,
                        c_int, P]),

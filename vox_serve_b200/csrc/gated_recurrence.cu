@@ -18,7 +18,7 @@
 // Real-gated linear recurrent unit (Griffin: De et al., "Griffin: Mixing Gated Linear Recurrences with Local Attention for
 // Efficient Language Models"):
 //   r_t = sigmoid(R_b u_t + br),  i_t = sigmoid(I_b u_t + bi)     in every block b of neighbouring channels, R_b, I_b square
-//   log a_t = -c r_t softplus(lam),  S_t = a_t S_(t-1) + sqrt(1 - a_t^2) i_t u_t,  out_t = S_t * gelu_tanh(y_t + by)
+//   log a_t = -rate r_t (rate = c softplus(lam)),  S_t = a_t S_(t-1) + sqrt(1 - a_t^2) i_t u_t,  out_t = S_t * gelu_tanh(y_t + by)
 //   vb_rglru         one kernel forms the gates of all rows (block-diagonal products: tensor cores for bf16 matrices whose
 //                    blocks are multiples of 16 channels, with u split into two bf16 terms so that a product keeps 16 bits of
 //                    u's mantissa; fp32 FMAs otherwise) and finishes the rows of requests that bring one row; the others leave
@@ -199,7 +199,7 @@ struct RgLruParams {
   int ld_u;
   const void* w;          // [blocks][2 * bs][bs]: the matrix of r, then that of i
   const float* bias;      // [blocks][2 * bs]
-  const float* lam;       // [C]
+  const float* rate;      // [C]: c * softplus(lam)
   const float* y;         // [T][ld_y]: the other branch before its bias and gelu
   int ld_y;
   const float* y_bias;    // [C] or nullptr
@@ -212,7 +212,6 @@ struct RgLruParams {
   const int32_t* pos;
   const int32_t* slots;
   int T, B, C, bs;
-  float c;
   int n_tiles, tile_rows; // piecewise form
   const int32_t* tile_req;
   const int32_t* tile_row0;
@@ -222,7 +221,6 @@ struct RgLruParams {
 __device__ __forceinline__ float gelu_tanh_f(float v) {
   return 0.5f * v * (1.f + tanhf(0.79788456080286536f * (v + 0.044715f * v * v * v)));
 }
-__device__ __forceinline__ float softplus_f(float v) { return fmaxf(v, 0.f) + log1pf(expf(-fabsf(v))); }
 
 template <typename CT>
 __device__ __forceinline__ void rg_out(const RgLruParams& p, int t, int ch, float S) {
@@ -233,7 +231,7 @@ __device__ __forceinline__ void rg_out(const RgLruParams& p, int t, int ch, floa
 // gate pre-activations zr, zi of (row, channel) -> the decay and scaled input; a request's only row is finished here
 template <typename CT>
 __device__ __forceinline__ void rg_finish(const RgLruParams& p, int t, int ch, float zr, float zi) {
-  const float la = -p.c * mg_sigmoid(zr) * softplus_f(p.lam[ch]);
+  const float la = -p.rate[ch] * mg_sigmoid(zr);
   const float a = expf(la);
   const float v = sqrtf(-expm1f(2.f * la)) * mg_sigmoid(zi) * p.u[static_cast<size_t>(t) * p.ld_u + ch];
   const int b = p.row_req[t];
@@ -387,13 +385,13 @@ __global__ void __launch_bounds__(128) rglru_gates_mma_kernel(RgLruParams p) {
   // as rg_finish, with all loads of a row's eight channels in flight before the first store
   const int lc = c0 + (lane & 3) * 2, gc = blk * p.bs + lc;
   const float* bias = p.bias + static_cast<size_t>(blk) * 2 * p.bs + lc;
-  float lam[4][2], br[4][2], bi[4][2];
+  float rate[4][2], br[4][2], bi[4][2];
 #pragma unroll
   for (int n = 0; n < 4; ++n)
 #pragma unroll
     for (int e = 0; e < 2; ++e) {
       const bool ok = lc + n * 8 < p.bs;
-      lam[n][e] = ok ? p.lam[gc + n * 8 + e] : 0.f;
+      rate[n][e] = ok ? p.rate[gc + n * 8 + e] : 0.f;
       br[n][e] = ok ? bias[n * 8 + e] : 0.f;
       bi[n][e] = ok ? bias[p.bs + n * 8 + e] : 0.f;
     }
@@ -423,7 +421,7 @@ __global__ void __launch_bounds__(128) rglru_gates_mma_kernel(RgLruParams p) {
       float a[2], v[2];
 #pragma unroll
       for (int e = 0; e < 2; ++e) {
-        const float la = -p.c * mg_sigmoid(acc[n][2 * half + e] + br[n][e]) * softplus_f(lam[n][e]);
+        const float la = -rate[n][e] * mg_sigmoid(acc[n][2 * half + e] + br[n][e]);
         a[e] = expf(la);
         v[e] = sqrtf(-expm1f(2.f * la)) * mg_sigmoid(acc[n + 4][2 * half + e] + bi[n][e]) * (e ? u[n].y : u[n].x);
       }
@@ -553,11 +551,11 @@ int vb_mingru_tiled(void* d_out, float* d_state, float* d_scratch, const float* 
 }
 
 int vb_rglru(void* d_out, int ld_out, float* d_state, float* d_ab, float* d_scratch, const float* d_u, int ld_u, const void* d_w,
-             const float* d_bias, const float* d_lam, float c, const float* d_y, int ld_y, const float* d_y_bias,
+             const float* d_bias, const float* d_rate, const float* d_y, int ld_y, const float* d_y_bias,
              const int32_t* d_qo_indptr, const int32_t* d_row_req, const int32_t* d_pos, const int32_t* d_slots,
              const int32_t* d_tile_req, const int32_t* d_tile_row0, int n_tiles, int tile_rows, int T, int B, int width,
              int blocks, int multi_rows, int w_dtype, int out_dtype, void* stream) {
-  VB_CHECK_ARG(d_out && d_state && d_u && d_w && d_bias && d_lam && d_y && d_qo_indptr && d_row_req && d_pos && d_slots &&
+  VB_CHECK_ARG(d_out && d_state && d_u && d_w && d_bias && d_rate && d_y && d_qo_indptr && d_row_req && d_pos && d_slots &&
                (!multi_rows || d_ab), "vb_rglru: null pointer");
   VB_CHECK_ARG(width > 0 && blocks > 0 && width % blocks == 0 && ld_u >= width && ld_y >= width && ld_out >= width,
                "vb_rglru: width %d in %d blocks", width, blocks);
@@ -565,8 +563,8 @@ int vb_rglru(void* d_out, int ld_out, float* d_state, float* d_ab, float* d_scra
                "vb_rglru: the piecewise form needs tiles of a multiple of %d rows and scratch", MG_ROWS);
   if (T <= 0 || B <= 0) return 0;
   const int bs = width / blocks;
-  RgLruParams p{d_u, ld_u, d_w, d_bias, d_lam, d_y, ld_y, d_y_bias, d_state, d_out, ld_out, d_ab, d_qo_indptr, d_row_req, d_pos,
-                d_slots, T, B, width, bs, c, n_tiles, tile_rows, d_tile_req, d_tile_row0, d_scratch};
+  RgLruParams p{d_u, ld_u, d_w, d_bias, d_rate, d_y, ld_y, d_y_bias, d_state, d_out, ld_out, d_ab, d_qo_indptr, d_row_req, d_pos,
+                d_slots, T, B, width, bs, n_tiles, tile_rows, d_tile_req, d_tile_row0, d_scratch};
   const bool f32 = out_dtype == 1;
   const dim3 grid(blocks * ((bs + RG_CH - 1) / RG_CH), (T + RG_R - 1) / RG_R);
   if (w_dtype == 0 && bs % 16 == 0 && ld_u % 4 == 0 && reinterpret_cast<uintptr_t>(d_u) % 16 == 0 && reinterpret_cast<uintptr_t>(d_w) % 16 == 0) {

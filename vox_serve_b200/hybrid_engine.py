@@ -747,11 +747,13 @@ class HybridWeights:
             bs = r.width // r.blocks
             ra, ri = mat(x + "right.ra"), mat(x + "right.ri")
             w["conv"], w["conv_b"] = vec(x + "right.conv"), vec(x + "right.conv.b")
-            w["y_b"], w["x_b"], w["lam"] = vec(x + "right.y.b"), vec(x + "right.x.b"), vec(x + "right.lam")
+            w["y_b"], w["x_b"] = vec(x + "right.y.b"), vec(x + "right.x.b")
+            lam = sd[x + "right.lam"].to(device=self.device, dtype=torch.float64)
+            w["rate"] = (r.c * (torch.clamp(lam, min=0.0) + torch.log1p(torch.exp(-lam.abs())))).to(F32).contiguous()
             w["left_norm"], w["right_norm"] = vec(x + "left.out"), vec(x + "right.out")
             if (any(tuple(t.shape) != (r.width, W) for t in (y, u)) or tuple(ro.shape) != (W, r.width) or
                     any(tuple(t.shape) != (r.blocks, bs, bs) for t in (ra, ri)) or tuple(w["conv"].shape) != (r.width, r.conv) or
-                    any(w[n].numel() != r.width for n in ("conv_b", "y_b", "x_b", "lam")) or
+                    any(w[n].numel() != r.width for n in ("conv_b", "y_b", "x_b", "rate")) or
                     any(w[n].numel() != W for n in ("left_norm", "right_norm"))):
                 raise VoxB200Error(f"layer {i}: gated linear recurrence shapes do not match the configuration")
             w["in"] = dense(torch.cat([qkv, y, u], 0).contiguous())
@@ -1885,7 +1887,7 @@ class HybridEngine:
         if (s.multi and s.tiles is not None and self.use_tiled_recurrence and
                 ops.mingru_scratch_floats(s.tiles[2], self.lin_tile_rows, C) <= self.glr_scratch.numel()):
             tiles = (*s.tiles, self.lin_tile_rows)
-        return ops.rglru(u, w["gates"], w["gates_b"], w["lam"], m.c, y, w["y_b"], cache.state[i], out, self.glr_ab, s.qo_indptr, s.row_req,
+        return ops.rglru(u, w["gates"], w["gates_b"], w["rate"], y, w["y_b"], cache.state[i], out, self.glr_ab, s.qo_indptr, s.row_req,
                          s.pos, s.slots, s.B, multi_rows=s.multi, tiles=tiles, scratch=self.glr_scratch)
 
     def _state_space(self, i: int, m: StateSpaceConfig, w: Dict[str, Any], s: StepInputs) -> torch.Tensor:

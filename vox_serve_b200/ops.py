@@ -1218,12 +1218,12 @@ def mingru_tiled(proj: torch.Tensor, z_off: int, x_off: int, g_off: int, bz: Opt
     return out
 
 
-def rglru(u: torch.Tensor, w: torch.Tensor, bias: torch.Tensor, lam: torch.Tensor, c: float, y: torch.Tensor,
+def rglru(u: torch.Tensor, w: torch.Tensor, bias: torch.Tensor, rate: torch.Tensor, y: torch.Tensor,
           y_bias: Optional[torch.Tensor], state: torch.Tensor, out: torch.Tensor, ab: Optional[torch.Tensor], qo_indptr: torch.Tensor,
           row_req: torch.Tensor, pos: torch.Tensor, slots: torch.Tensor, B: int, multi_rows: bool = True,
           tiles: Optional[Tuple[torch.Tensor, torch.Tensor, int, int]] = None, scratch: Optional[torch.Tensor] = None) -> torch.Tensor:
     """Real-gated linear recurrent unit: r = sigmoid(R_b u + br), i = sigmoid(I_b u + bi) per block b of neighbouring channels,
-    log a = -c r softplus(lam), S_t = a S_(t-1) + sqrt(1 - a^2) i u, out = S * gelu_tanh(y + y_bias).  u, y: fp32 views [T, C];
+    log a = -rate r (fp32 [C]: c * softplus of the stored parameter), S_t = a S_(t-1) + sqrt(1 - a^2) i u, out = S * gelu_tanh(y + y_bias).  u, y: fp32 views [T, C];
     w [blocks, 2 * C / blocks, C / blocks] (R_b above I_b; bf16 or fp32), bias fp32 [blocks, 2 * C / blocks]; state fp32
     [slots, C] (taken as zero where a request starts at position 0); out a view [T, C] (bf16 or fp32).  multi_rows: some request
     brings several rows (ab: fp32 scratch of 2 T C); tiles = (tile_req, tile_row0, n_tiles, tile_rows) + scratch: those in
@@ -1233,7 +1233,7 @@ def rglru(u: torch.Tensor, w: torch.Tensor, bias: torch.Tensor, lam: torch.Tenso
     blocks, bs = w.shape[0], w.shape[2]
     assert u.dtype == F32 and u.stride(1) == 1 and y.dtype == F32 and y.stride(1) == 1 and tuple(y.shape) == (T, C)
     assert w.is_contiguous() and w.shape[1] == 2 * bs and blocks * bs == C and bias.dtype == F32 and bias.numel() == 2 * C
-    assert lam.dtype == F32 and lam.numel() == C and (y_bias is None or (y_bias.dtype == F32 and y_bias.numel() == C))
+    assert rate.dtype == F32 and rate.numel() == C and (y_bias is None or (y_bias.dtype == F32 and y_bias.numel() == C))
     assert state.dtype == F32 and state.is_contiguous() and state.shape[1] == C and out.stride(1) == 1 and tuple(out.shape) == (T, C)
     assert not multi_rows or (ab is not None and ab.dtype == F32 and ab.numel() >= 2 * T * C)
     tr = t0 = None
@@ -1243,7 +1243,7 @@ def rglru(u: torch.Tensor, w: torch.Tensor, bias: torch.Tensor, lam: torch.Tenso
         tr, t0 = tile_req.data_ptr(), tile_row0.data_ptr()
         assert scratch is not None and scratch.dtype == F32 and scratch.numel() >= mingru_scratch_floats(n_tiles, tile_rows, C)
     call("vb_rglru", out.data_ptr(), out.stride(0), state.data_ptr(), _p(ab), _p(scratch), u.data_ptr(), u.stride(0), w.data_ptr(),
-         bias.data_ptr(), lam.data_ptr(), float(c), y.data_ptr(), y.stride(0), _p(y_bias), qo_indptr.data_ptr(), row_req.data_ptr(),
+         bias.data_ptr(), rate.data_ptr(), y.data_ptr(), y.stride(0), _p(y_bias), qo_indptr.data_ptr(), row_req.data_ptr(),
          pos.data_ptr(), slots.data_ptr(), tr, t0, n_tiles, tile_rows, T, B, C, blocks, int(multi_rows), _dt(w), _dt(out), _stream())
     if multi_rows:
         _lib.launch_counter[0] += 3 if n_tiles else 1      # (beside the one that ``call`` counts)
